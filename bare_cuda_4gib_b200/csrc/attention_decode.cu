@@ -155,6 +155,7 @@ struct DecodeArgs {
   const int32_t* tile_index;
   float scale_log2;
   int window;
+  AttentionExtras extras;
   int* error_word;
 };
 
@@ -203,7 +204,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
   const int last_token = min(q_len - 1, (row0 + BM - 1) / group), first_token = row0 / group;
   const int hi_key = pos0 + last_token;
   const int tile_min_pos = pos0 + first_token, tile_max_pos = pos0 + last_token;
-  const int lo_key = a.window > 0 ? max(0, pos0 + first_token - a.window + 1) : 0;
+  const int lo_key = first_visible_key(tile_min_pos, a.window, a.extras.chunk);
+  const int tile_max_lo = first_visible_key(tile_max_pos, a.window, a.extras.chunk);   // from here on no row's bound hides a key
   const int kb_lo = lo_key / BN, kb_hi = hi_key / BN;   // inclusive
   // this warp's key blocks: kb_lo + gw, kb_lo + gw + stride, ...
   const int stride = WARPS * n_splits, gw = split * WARPS + warp;
@@ -282,12 +284,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
   for (int ks = 0; ks < D / 16; ++ks)
     ldmatrix_x4(qf[ks], smem_u32(Qs + (lane & 15) * QLD + ks * 16 + (lane >> 4) * 8));
 
-  int row_pos[2];
+  int row_pos[2], row_lo[2];
   float m[2], l[2], o[D / 8][4];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int R = row0 + (lane >> 2) + h * 8;
     row_pos[h] = R < n_rows ? pos0 + R / group : -1;
+    row_lo[h] = first_visible_key(row_pos[h], a.window, a.extras.chunk);
     m[h] = -INFINITY;
     l[h] = 0.0f;
   }
@@ -319,7 +322,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
       }
     }
 
-    const bool all_visible = key0 + BN - 1 <= tile_min_pos && (a.window <= 0 || key0 > tile_max_pos - a.window);
+    const bool all_visible = key0 + BN - 1 <= tile_min_pos && key0 >= tile_max_lo;
     float mx[2] = {-INFINITY, -INFINITY};
     if (all_visible) {
 #pragma unroll
@@ -337,7 +340,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
         for (int e = 0; e < 4; ++e) {
           const int h = e >> 1;
           const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-          const bool visible = key <= row_pos[h] && (a.window <= 0 || key > row_pos[h] - a.window);
+          const bool visible = key <= row_pos[h] && key >= row_lo[h];
           const float v = visible ? s[nt][e] * a.scale_log2 : -INFINITY;
           s[nt][e] = v;
           mx[h] = fmaxf(mx[h], v);
@@ -449,9 +452,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
     const int slot = i / (D / 4), c4 = i % (D / 4);
     const int r = slot * n_splits + split, R = row0 + r;
     if (r >= BM || R >= n_rows) continue;
-    float M = -INFINITY;
+    const int token = R / group, head = kvh * group + R % group;
+    const float sink = sink_log2(a.extras, head);     // joins the row's sum here, once
+    float M = sink;
     for (int z = 0; z < n_splits; ++z) M = fmaxf(M, recv[((size_t)z * owned_rows + slot) * STATE + D]);
-    float L = 0.0f;
+    float L = M != -INFINITY ? exp2f(sink - M) : 0.0f;
     float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (M != -INFINITY) {
       for (int z = 0; z < n_splits; ++z) {
@@ -465,8 +470,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
         acc.w += v.w * f;
       }
     }
-    const float inv = L > 0.0f ? 1.0f / L : 0.0f;
-    const int token = R / group, head = kvh * group + R % group;
+    const float inv = L > 0.0f ? head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / L : 0.0f;
     uint2 packed;
     packed.x = pack_bf16(acc.x * inv, acc.y * inv);
     packed.y = pack_bf16(acc.z * inv, acc.w * inv);
@@ -522,14 +526,15 @@ extern "C" int llm_attention_decode_pool_map(void* map_out, const void* base, lo
 // Tiles of 16 packed rows (the tile list of llm_attention_mma's decode shape).  `n_splits` blocks
 // (1..8) share a tile's key blocks as one cluster; `slots` (1..3) key blocks per warp are in
 // flight.  `pool_map`: llm_attention_decode_pool_map over `pool_base`, in which k_base and v_base
-// lie, with boxes of `box_rows` rows (a multiple of 8 that divides 64 and the page size).
+// lie, with boxes of `box_rows` rows (a multiple of 8 that divides 64 and the page size).  chunk, sink, gate and
+// gate_stride (elements): `AttentionExtras`; 0 and null: none.
 extern "C" int llm_attention_decode(const void* pool_map, const void* pool_base, long long pool_rows, int box_rows,
                                     const void* q, void* out, void* k_base, void* v_base, const int32_t* block_table,
                                     long long page_stride, int table_stride, int page_tokens, int kv_heads,
                                     int head_dim, const int32_t* seq_q_start, const int32_t* seq_q_len,
                                     const int32_t* seq_kv_len, const int32_t* tile_seq, const int32_t* tile_index,
                                     int n_tiles, int n_splits, int slots, int q_heads, float scale, int window,
-                                    int* error_word, cudaStream_t stream) {
+                                    int chunk, const float* sink, const void* gate, long long gate_stride, int* error_word, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (head_dim != D || q_heads % kv_heads || kv_heads > 65535 || n_splits < 1 || n_splits > 8 || slots < 1 ||
       slots > MAX_SLOTS)
@@ -560,6 +565,7 @@ extern "C" int llm_attention_decode(const void* pool_map, const void* pool_base,
   a.tile_seq = tile_seq, a.tile_index = tile_index;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.window = window;
+  a.extras = AttentionExtras{chunk, sink, gate, gate_stride};
   a.error_word = error_word;
 
   cudaLaunchConfig_t cfg = {};

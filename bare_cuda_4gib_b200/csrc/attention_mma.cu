@@ -34,6 +34,8 @@
 // -DV_DIM=n builds the kernel for value heads of n entries beside key heads of HEAD_DIM (a multiple of 16 up
 // to 128; default: HEAD_DIM).  -DSCORE_CAP builds the variant whose scaled score s becomes cap * tanh(s / cap)
 // before the softmax (entry point `llm_attention_mma_general`, which every build has for its value size).
+// That entry point also takes `AttentionExtras` (common.cuh): blocks of positions, a sink per head, which
+// joins the sum where a row is finished, and a sigmoid gate per head on the way out.
 
 #include "common.cuh"
 
@@ -120,6 +122,7 @@ struct AttnArgs {
   int bias_len;
   float scale_over_cap;        // SCORE_CAP: scale / cap, and cap * log2(e)
   float cap_log2;
+  AttentionExtras extras;
 };
 
 // SCORE_CAP: what a raw score q . k becomes, in base-2 units: cap * tanh(score * scale / cap) * log2(e), with
@@ -169,8 +172,8 @@ attention_mma_kernel(AttnArgs a) {
   // (their queries are zero, their scores finite).
   const int tile_min_pos = pos0 + first_token;
   const int tile_max_pos = pos0 + last_token;
-  int lo_key = 0;
-  if (a.window > 0) lo_key = max(0, pos0 + first_token - a.window + 1);
+  const int lo_key = first_visible_key(tile_min_pos, a.window, a.extras.chunk);
+  const int tile_max_lo = first_visible_key(tile_max_pos, a.window, a.extras.chunk);   // from here on no row's bound hides a key
   const int kb_lo = lo_key / BN, kb_hi = hi_key / BN;  // inclusive
   const int n_kb_total = kb_hi - kb_lo + 1;
   const int per_split = (n_kb_total + n_splits - 1) / n_splits;
@@ -271,7 +274,7 @@ attention_mma_kernel(AttnArgs a) {
       ldmatrix_x4(qf[mt][ks], Qs + (wm * WR + mt * 16 + (lane & 15)) * LDS + ks * 16 + (lane >> 4) * 8);
 
   // this thread's rows: two per row tile
-  int row_pos[MT][2];
+  int row_pos[MT][2], row_lo[MT][2];
 #ifdef DISTANCE_BIAS
   const float* row_bias[MT][2];  // the bias row of this row's head
 #endif
@@ -283,6 +286,7 @@ attention_mma_kernel(AttnArgs a) {
     for (int h = 0; h < 2; ++h) {
       const int R = row0 + wm * WR + mt * 16 + (lane >> 2) + h * 8;
       row_pos[mt][h] = R < n_rows ? pos0 + R / group : -1;  // -1: no key is visible
+      row_lo[mt][h] = first_visible_key(row_pos[mt][h], a.window, a.extras.chunk);
 #ifdef DISTANCE_BIAS
       row_bias[mt][h] = a.bias + (long long)(kvh * group + R % group) * a.bias_len;
 #endif
@@ -327,7 +331,7 @@ attention_mma_kernel(AttnArgs a) {
     const bool all_visible = false;   // every score gets its own bias: one path
     uint32_t pf_lo[MT][NT / 2][4];
 #else
-    const bool all_visible = kb * BN + BN - 1 <= tile_min_pos && (a.window <= 0 || kb * BN > tile_max_pos - a.window);
+    const bool all_visible = kb * BN + BN - 1 <= tile_min_pos && kb * BN >= tile_max_lo;
 #endif
     uint32_t pf[MT][NT / 2][4];
 #pragma unroll
@@ -355,7 +359,7 @@ attention_mma_kernel(AttnArgs a) {
           for (int e = 0; e < 4; ++e) {
             const int h = e >> 1;
             const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-            const bool visible = key <= row_pos[mt][h] && (a.window <= 0 || key > row_pos[mt][h] - a.window);
+            const bool visible = key <= row_pos[mt][h] && key >= row_lo[mt][h];
 #ifdef DISTANCE_BIAS
             const float v = visible ? fmaf(s[mt][nt][e], a.scale_log2,
                                            1.4426950408889634f * __ldg(row_bias[mt][h] + min(row_pos[mt][h] - key, a.bias_len - 1)))
@@ -463,10 +467,13 @@ attention_mma_kernel(AttnArgs a) {
   for (int i = threadIdx.x; i < BM * CHUNKS_V; i += NT_THREADS) {
     const int r = i / CHUNKS_V, c = i % CHUNKS_V;
     const int R = row0 + r;
-    float M = -INFINITY;
+    const int token = R / group, head = kvh * group + R % group;
+    // a row that is finished here (keys not split) has the sink in its sum from the start
+    const float sink = n_splits == 1 && R < n_rows ? sink_log2(a.extras, head) : -INFINITY;
+    float M = sink;
 #pragma unroll
     for (int w = 0; w < WARPS_N; ++w) M = fmaxf(M, red_m[w * BM + r]);
-    float L = 0.0f, acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+    float L = M != -INFINITY ? exp2f(sink - M) : 0.0f, acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
     if (M != -INFINITY) {
 #pragma unroll
       for (int w = 0; w < WARPS_N; ++w) {
@@ -477,10 +484,9 @@ attention_mma_kernel(AttnArgs a) {
         for (int e = 0; e < 8; ++e) acc[e] += src[e] * f;
       }
     }
-    const float inv = L > 0.0f ? (n_splits == 1 ? a.out_scale : 1.0f) / L : 0.0f;
     if (n_splits == 1) {
       if (R < n_rows) {
-        const int token = R / group, head = kvh * group + R % group;
+        const float inv = L > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / L : 0.0f;
         uint4 packed;
         packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
         packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
@@ -489,6 +495,7 @@ attention_mma_kernel(AttnArgs a) {
         *reinterpret_cast<uint4*>(a.out + (long long)(q_start + token) * a.out_stride + head * DV + c * 8) = packed;
       }
     } else {
+      const float inv = L > 0.0f ? 1.0f / L : 0.0f;
       float* dst = a.part_o + (item * BM + r) * DV + c * 8;
 #pragma unroll
       for (int e = 0; e < 8; ++e) dst[e] = acc[e] * inv;
@@ -521,9 +528,11 @@ attention_mma_kernel(AttnArgs a) {
     const int R = row0 + r;
     if (R >= n_rows) continue;
     auto lse_at = [&](int z) { return lse_fits ? lse[z * BM + r] : __ldcg(a.part_lse + (item0 + z) * BM + r); };
-    float M = -INFINITY;
+    const int token = R / group, head = kvh * group + R % group;
+    const float sink = sink_log2(a.extras, head);
+    float M = sink;
     for (int z = 0; z < n_splits; ++z) M = fmaxf(M, lse_at(z));
-    float W = 0.0f, acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+    float W = M != -INFINITY ? exp2f(sink - M) : 0.0f, acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
     if (M != -INFINITY) {
 #pragma unroll 4
       for (int z = 0; z < n_splits; ++z) {   // independent loads: several are in flight at once
@@ -535,8 +544,7 @@ attention_mma_kernel(AttnArgs a) {
         acc[4] += w * hi.x; acc[5] += w * hi.y; acc[6] += w * hi.z; acc[7] += w * hi.w;
       }
     }
-    const float inv = W > 0.0f ? a.out_scale / W : 0.0f;
-    const int token = R / group, head = kvh * group + R % group;
+    const float inv = W > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / W : 0.0f;
     uint4 packed;
     packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
     packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
@@ -598,7 +606,8 @@ static int attention_mma_launch(const void* q, void* out, long long out_stride, 
                                 int head_dim, const int32_t* seq_q_start, const int32_t* seq_q_len,
                                 const int32_t* seq_kv_len, const int32_t* tile_seq, const int32_t* tile_index,
                                 int n_tiles, int rows_per_tile, int n_splits, float* scratch, int q_heads,
-                                float scale, int window, cudaStream_t stream, float cap = 0.0f) {
+                                float scale, int window, cudaStream_t stream, float cap = 0.0f,
+                                AttentionExtras extras = AttentionExtras{0, nullptr, nullptr, 0}) {
   if (n_tiles <= 0) return 0;
   if (out_stride % 8) return ERR_BAD_ALIGN;
 #ifdef SCORE_CAP
@@ -633,6 +642,7 @@ static int attention_mma_launch(const void* q, void* out, long long out_stride, 
   a.bias_len = bias_len;
   a.scale_over_cap = cap > 0.0f ? scale / cap : 0.0f;
   a.cap_log2 = cap * 1.4426950408889634f;
+  a.extras = extras;
   if (rows_per_tile == 64 * PREFILL_MT) return launch<4, 1, PREFILL_MT>(a, n_tiles, kv_heads, n_splits, stream);
   if (rows_per_tile == 16) return launch<1, 4, 1>(a, n_tiles, kv_heads, n_splits, stream);
   return ERR_BAD_SIZE;
@@ -658,18 +668,20 @@ extern "C" int llm_attention_mma(const void* q, void* out, void* k_base, void* v
 
 #ifndef DISTANCE_BIAS
 // Value heads of `v_dim` entries (this library's V_DIM) beside key heads of `head_dim`, and `cap` (0: none; a
-// library built with -DSCORE_CAP takes a positive one): score <- cap * tanh(score * scale / cap).
+// library built with -DSCORE_CAP takes a positive one): score <- cap * tanh(score * scale / cap).  chunk, sink,
+// gate and gate_stride (elements): `AttentionExtras`; 0 and null: none.
 extern "C" int llm_attention_mma_general(const void* q, void* out, void* k_base, void* v_base, const int32_t* block_table,
                                          long long page_stride, int table_stride, int page_tokens, int kv_heads,
                                          int head_dim, int v_dim, const int32_t* seq_q_start, const int32_t* seq_q_len,
                                          const int32_t* seq_kv_len, const int32_t* tile_seq, const int32_t* tile_index,
                                          int n_tiles, int rows_per_tile, int n_splits, float* scratch, int q_heads,
-                                         float scale, int window, float cap, cudaStream_t stream) {
+                                         float scale, int window, float cap, int chunk, const float* sink, const void* gate,
+                                         long long gate_stride, cudaStream_t stream) {
   if (v_dim != DV) return ERR_BAD_SIZE;
   return attention_mma_launch(q, out, (long long)q_heads * DV, 1.0f, nullptr, 0, k_base, v_base, block_table, page_stride,
                               table_stride, page_tokens, kv_heads, head_dim, seq_q_start, seq_q_len, seq_kv_len,
                               tile_seq, tile_index, n_tiles, rows_per_tile, n_splits, scratch, q_heads, scale, window,
-                              stream, cap);
+                              stream, cap, AttentionExtras{chunk, sink, gate, gate_stride});
 }
 #endif
 

@@ -212,6 +212,7 @@ struct AttnArgs {
   int q_heads;
   float scale_log2;
   int window;
+  AttentionExtras extras;
   int* error_word;
 };
 
@@ -268,7 +269,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
       const int first_token = first_row / group, last_token = min(q_len - 1, (first_row + BM - 1) / group);
       g_min_pos[g] = pos0 + first_token;
       g_max_pos[g] = pos0 + last_token;
-      const int lo_key = a.window > 0 ? max(0, g_min_pos[g] - a.window + 1) : 0;
+      const int lo_key = first_visible_key(g_min_pos[g], a.window, a.extras.chunk);
       g_lo[g] = lo_key / BN;
       g_hi[g] = g_max_pos[g] / BN + 1;
       lo_all = min(lo_all, g_lo[g]);
@@ -506,7 +507,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
     const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
     const uint32_t s_addr = lane_addr + g * BN, o_addr = lane_addr + O_COL + g * D;
     const int my_lo = g_lo[g], my_n = g_hi[g] - g_lo[g];
-    const int tile_min_pos = g_min_pos[g], tile_max_pos = g_max_pos[g];
+    const int row_lo = first_visible_key(row_pos, a.window, a.extras.chunk);
+    const int tile_min_pos = g_min_pos[g];
+    const int tile_max_lo = first_visible_key(g_max_pos[g], a.window, a.extras.chunk);   // from here on no row's bound hides a key
     // Running softmax of the row.  `m` is the maximum the exponentials are taken against; it follows the
     // true maximum only when that has grown by more than RESCALE_STEP (in base-2 units), so that O, which
     // accumulates in tensor memory over all key blocks, has to be rescaled rarely: with a stale maximum
@@ -524,7 +527,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
       ok = mbar_wait(&s_full[g], i & 1, abort_flag) && !*abort_flag;
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const bool all_visible = key0 + BN - 1 <= tile_min_pos && (a.window <= 0 || key0 > tile_max_pos - a.window);
+      const bool all_visible = key0 + BN - 1 <= tile_min_pos && key0 >= tile_max_lo;
       // The row of S is read once, in two pieces of 64 columns (one sub-tile of P each).  Each piece
       // settles the maximum for itself: should the second piece move it, the probabilities of the
       // first, which this thread has just written, are rescaled where they lie (rare, as is every move).
@@ -543,7 +546,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
 #pragma unroll
           for (int k = 0; k < S_PIECE; ++k) {
             const int key = key0 + h * S_PIECE + k;
-            const bool visible = key <= row_pos && (a.window <= 0 || key > row_pos - a.window);
+            const bool visible = key <= row_pos && key >= row_lo;
             if (!visible) v[k] = 0xff800000u;   // -inf: probability 0
           }
         }
@@ -633,8 +636,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
     // rows do in the tile.  (The loads are warp-wide, so rows without an output still take part.)
     if (ok && my_n > 0) {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const float inv = l > 0.0f ? 1.0f / l : 0.0f;
       const int token = row_valid ? R / group : 0, head = row_valid ? kvh * group + R % group : 0;
+      // the sink joins the sum, taken against the same maximum (far above it the sum is infinite, the row zero)
+      if (a.extras.sink && row_valid) l += exp2f(sink_log2(a.extras, head) - m);
+      const float inv = l > 0.0f ? (row_valid ? head_gate<__nv_bfloat16>(a.extras, q_start + token, head) : 1.0f) / l : 0.0f;
       uint4* dst = reinterpret_cast<uint4*>(a.out + ((long long)(q_start + token) * a.q_heads + head) * D);
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 32) {
@@ -700,14 +705,15 @@ extern "C" int llm_attention_tc_rows() { return BLOCK_ROWS; }
 // Same arguments as llm_attention_mma without splits and scratch, plus the pool's tensor map
 // (llm_attention_tc_pool_map over `pool_base`, which k_base and v_base lie in, with boxes of
 // `box_rows` rows: a multiple of 8 that divides both 128 and the page size).  Every tile has 256
-// packed rows (llm_attention_tc_rows).
+// packed rows (llm_attention_tc_rows).  chunk, sink, gate and gate_stride (elements): `AttentionExtras`; 0 and
+// null: none.
 extern "C" int llm_attention_tcgen05(const void* pool_map, const void* pool_base, int box_rows, const void* q, void* out,
                                      void* k_base, void* v_base, const int32_t* block_table,
                                      long long page_stride, int table_stride, int page_tokens, int kv_heads,
                                      int head_dim, const int32_t* seq_q_start, const int32_t* seq_q_len,
                                      const int32_t* seq_kv_len, const int32_t* tile_seq, const int32_t* tile_index,
-                                     int n_tiles, int q_heads, float scale, int window, int* error_word,
-                                     cudaStream_t stream) {
+                                     int n_tiles, int q_heads, float scale, int window, int chunk, const float* sink,
+                                     const void* gate, long long gate_stride, int* error_word, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (head_dim != D || q_heads % kv_heads || kv_heads > 65535) return ERR_BAD_SIZE;
   if (box_rows < 8 || box_rows % 8 || BN % box_rows || page_tokens % box_rows) return ERR_BAD_SIZE;
@@ -742,6 +748,7 @@ extern "C" int llm_attention_tcgen05(const void* pool_map, const void* pool_base
   a.q_heads = q_heads;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.window = window;
+  a.extras = AttentionExtras{chunk, sink, gate, gate_stride};
   a.error_word = error_word;
   if (n_tiles > 65535) return ERR_BAD_SIZE;
   dim3 grid(kv_heads, n_tiles);

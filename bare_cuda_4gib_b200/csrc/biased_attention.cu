@@ -175,14 +175,14 @@ extern "C" int llm_conv_ring_write(const void* u, int dtype, long long u_stride,
 // One warp per (row, query head).  Keys are walked in blocks of 32 absolute positions (block b
 // holds positions 32 b .. 32 b + 31), one key per lane: score = (q . k) * scale +
 // bias[head][distance] (with `softcap` > 0 the scaled score first becomes softcap * tanh(score / softcap));
-// online softmax over blocks; the value sum with one output channel group
+// online softmax over blocks, `extras` as AttentionExtras says; the value sum with one output channel group
 // per lane.  Each sum's order depends on the sizes and on absolute key positions only.
 template <typename T>
 __global__ void __launch_bounds__(BA_WARPS * 32)
 biased_attention_kernel(const T* __restrict__ q, T* __restrict__ out, long long out_stride, PagedCacheKV cache,
                         const float* __restrict__ bias, int bias_len, const int32_t* __restrict__ positions,
                         const int32_t* __restrict__ row_seq, int q_heads, int n_tokens, float scale, int window,
-                        float out_scale, float softcap) {
+                        float out_scale, float softcap, AttentionExtras extras) {
   pdl_launch_dependents();
   extern __shared__ float q_sm[];   // [BA_WARPS][k_dim]
   const int dk = cache.k_dim, dv = cache.v_dim;
@@ -196,7 +196,7 @@ biased_attention_kernel(const T* __restrict__ q, T* __restrict__ out, long long 
   float* qs = q_sm + warp * dk;
   for (int d = lane; d < dk; d += 32) qs[d] = to_float(q[(long long)t * q_heads * dk + (long long)h * dk + d]);
   __syncwarp();
-  const int first = window > 0 ? max(0, p - window + 1) : 0;
+  const int first = first_visible_key(p, window, extras.chunk);
   const float* bias_h = bias ? bias + (long long)h * bias_len : nullptr;
   float m = -INFINITY, l = 0.0f;
   float acc[8];                      // value channels lane, lane + 32, ... (v_dim <= 256)
@@ -238,7 +238,13 @@ biased_attention_kernel(const T* __restrict__ q, T* __restrict__ out, long long 
       }
     }
   }
-  const float inv = l > 0.0f ? out_scale / l : 0.0f;
+  float from_sum = 1.0f;       // what the sums taken against m become against the maximum with the sink
+  if (extras.sink) {
+    const float s = extras.sink[h], m_new = fmaxf(m, s);
+    from_sum = m == -INFINITY ? 0.0f : expf(m - m_new);
+    l = l * from_sum + expf(s - m_new);
+  }
+  const float inv = l > 0.0f ? out_scale * from_sum * head_gate<T>(extras, t, h) / l : 0.0f;
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     const int d = lane + 32 * j;
@@ -250,22 +256,24 @@ extern "C" int llm_biased_attention(const void* q, void* out, int dtype, long lo
                                     void* cache_v, const int32_t* block_table, long long page_stride, int table_stride,
                                     int page_tokens, int kv_heads, int k_dim, int v_dim, const float* bias, int bias_len,
                                     const int32_t* positions, const int32_t* row_seq, int q_heads, int n_tokens,
-                                    float scale, int window, float out_scale, float softcap, cudaStream_t stream) {
+                                    float scale, int window, float out_scale, float softcap, int chunk, const float* sink,
+                                    const void* gate, long long gate_stride, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   LLM_HOST_CHECK(v_dim <= 256 && k_dim >= 1 && kv_heads >= 1 && q_heads % kv_heads == 0, ERR_BAD_SIZE);
   LLM_HOST_CHECK(bias == nullptr || bias_len >= 1, ERR_BAD_SIZE);
   const size_t smem = (size_t)BA_WARPS * k_dim * sizeof(float);
   LLM_HOST_CHECK(smem <= 48 * 1024, ERR_BAD_SIZE);
   PagedCacheKV cache{cache_k, cache_v, block_table, page_stride, table_stride, page_tokens, kv_heads, k_dim, v_dim};
+  const AttentionExtras extras{chunk, sink, gate, gate_stride};
   const long long items = (long long)n_tokens * q_heads;
   const int blocks = (int)((items + BA_WARPS - 1) / BA_WARPS);
   if (dtype == DT_F32)
     launch_kernel(biased_attention_kernel<float>, blocks, BA_WARPS * 32, smem, stream, (const float*)q, (float*)out,
-                  out_stride, cache, bias, bias_len, positions, row_seq, q_heads, n_tokens, scale, window, out_scale, softcap);
+                  out_stride, cache, bias, bias_len, positions, row_seq, q_heads, n_tokens, scale, window, out_scale, softcap, extras);
   else if (dtype == DT_BF16)
     launch_kernel(biased_attention_kernel<__nv_bfloat16>, blocks, BA_WARPS * 32, smem, stream, (const __nv_bfloat16*)q,
                   (__nv_bfloat16*)out, out_stride, cache, bias, bias_len, positions, row_seq, q_heads, n_tokens, scale,
-                  window, out_scale, softcap);
+                  window, out_scale, softcap, extras);
   else
     return ERR_BAD_DTYPE;
   return launch_status();

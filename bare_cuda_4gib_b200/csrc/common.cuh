@@ -6,6 +6,7 @@
 
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+#include <math.h>
 #include <stdint.h>
 #include <stdlib.h>
 
@@ -134,6 +135,38 @@ struct PagedCache {
   int kv_heads;
   int head_dim;
 };
+
+// What a softmax-attention kernel may be given beside its queries and its cache (all zero: none of it).
+// `chunk` > 0: a query sees the keys of its own block of `chunk` positions only, blocks counted from
+// position 0 of the sequence.  `sink` [q_heads] float32: exp(sink[head]) joins the softmax's denominator,
+// once, unscaled and without a value.  `gate` (the step's element type, row t of the step at t *
+// gate_stride): head h's output is multiplied by sigmoid(gate[t][h]).
+struct AttentionExtras {
+  int chunk;
+  const float* sink;
+  const void* gate;
+  long long gate_stride;
+};
+
+// The oldest position that a query at `pos` sees (window <= 0, chunk <= 0: no such bound).
+__device__ __forceinline__ int first_visible_key(int pos, int window, int chunk) {
+  int lo = 0;
+  if (window > 0) lo = max(lo, pos - window + 1);
+  if (chunk > 0) lo = max(lo, pos - pos % chunk);
+  return lo;
+}
+
+// The factor of head `head` in row `row` of the step.
+template <typename T>
+__device__ __forceinline__ float head_gate(const AttentionExtras& x, long long row, int head) {
+  if (!x.gate) return 1.0f;
+  return 1.0f / (1.0f + expf(-to_float(reinterpret_cast<const T*>(x.gate)[row * x.gate_stride + head])));
+}
+
+// The sink's share in base-2 units, sink[head] * log2(e); -inf without a sink.
+__device__ __forceinline__ float sink_log2(const AttentionExtras& x, int head) {
+  return x.sink ? x.sink[head] * 1.4426950408889634f : -INFINITY;
+}
 
 // Element offset of (batch sequence, position, kv head) inside the pool, or -1 if the page is not held.
 __device__ __forceinline__ long long cache_offset(const PagedCache& c, int seq, int pos, int kvh) {

@@ -9,6 +9,8 @@
 // (the maps of differential attention), each normed and turned by itself; the values belong to the head.  q goes
 // to its buffer, k into the request's cache page, and the values - a projection of their own, or
 // the keys as projected, before norm and rotation - beside it.  Grid (token, share of the token's heads).  Norm, angle and rotation are float32.
+// With `unit_norm` q and k are normed without a weight, rms_norm(rotate(x)): a rotation (mag 1) leaves the
+// root mean square of a head as it is, so the factor is formed from the entries as they are read.
 // `bias` (float32, indexed by the projection's column, or null) is added to q, k and v as they are read.
 // Value mixing: with `v_mix_in` [tokens, kv_heads * v_dim] float32 the value becomes (1 - v_mix) v + v_mix *
 // v_mix_in (another layer's values of the same token), and with `v_mix_out` the value as cached is also
@@ -24,7 +26,7 @@
 template <typename T, typename TW>
 __global__ void __launch_bounds__(PREP_WARPS * 32)
 headnorm_rope_cache_kernel(const T* __restrict__ u, long long u_stride, int q_col, int k_col, int v_col,
-                           const TW* __restrict__ q_norm_w, const TW* __restrict__ k_norm_w, float eps,
+                           const TW* __restrict__ q_norm_w, const TW* __restrict__ k_norm_w, int unit_norm, float eps,
                            const float* __restrict__ inv_freq, int rot_dims, int halves, int maps, float mag,
                            T* __restrict__ q_out, PagedCache cache, int v_dim, const int32_t* __restrict__ positions,
                            const int32_t* __restrict__ row_seq, int q_heads, int write_cache,
@@ -79,7 +81,7 @@ headnorm_rope_cache_kernel(const T* __restrict__ u, long long u_stride, int q_co
       s[c] = v;
       sq += v * v;
     }
-    const float scale = w ? 1.0f / sqrtf(warp_sum(sq) / (float)d + eps) : 1.0f;
+    const float scale = w || unit_norm ? 1.0f / sqrtf(warp_sum(sq) / (float)d + eps) : 1.0f;
     __syncwarp();
     const int half = rot_dims / 2;
     for (int p = lane; p < half; p += 32) {
@@ -100,7 +102,8 @@ headnorm_rope_cache_kernel(const T* __restrict__ u, long long u_stride, int q_co
 
 // dtype: element type of u, q_out, the cache and the norm weights.
 extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_stride, int q_col, int k_col, int v_col,
-                                       const void* q_norm_w, const void* k_norm_w, float eps, const float* inv_freq,
+                                       const void* q_norm_w, const void* k_norm_w, int unit_norm, float eps,
+                                       const float* inv_freq,
                                        int rot_dims, int halves, int maps, float mag, void* q_out, void* k_base,
                                        void* v_base,
                                        const int32_t* block_table, long long page_stride, int table_stride,
@@ -112,6 +115,7 @@ extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_str
   LLM_HOST_CHECK(maps >= 1 && head_dim % maps == 0, ERR_BAD_SIZE);
   LLM_HOST_CHECK(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= head_dim / maps && (rot_dims == 0 || inv_freq), ERR_BAD_SIZE);
   LLM_HOST_CHECK(v_col >= 0 || (v_dim == head_dim && maps == 1), ERR_BAD_SIZE);
+  LLM_HOST_CHECK(!unit_norm || (!q_norm_w && !k_norm_w && mag == 1.0f), ERR_BAD_SIZE);
   const size_t smem = (size_t)PREP_WARPS * head_dim * sizeof(float);
   LLM_HOST_CHECK(smem <= 48 * 1024, ERR_BAD_SIZE);
   PagedCache c{k_base, v_base, block_table, page_stride, table_stride, page_tokens, kv_heads, head_dim};
@@ -120,13 +124,13 @@ extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_str
   const dim3 grid(n_tokens, per_token);
   if (dtype == DT_F32)
     launch_kernel(headnorm_rope_cache_kernel<float, float>, grid, PREP_WARPS * 32, smem, stream, (const float*)u,
-                  u_stride, q_col, k_col, v_col, (const float*)q_norm_w, (const float*)k_norm_w, eps, inv_freq, rot_dims,
+                  u_stride, q_col, k_col, v_col, (const float*)q_norm_w, (const float*)k_norm_w, unit_norm, eps, inv_freq, rot_dims,
                   halves, maps, mag, (float*)q_out, c, v_dim, positions, row_seq, q_heads, write_cache, bias, v_mix_in, v_mix,
                   v_mix_out);
   else if (dtype == DT_BF16)
     launch_kernel(headnorm_rope_cache_kernel<__nv_bfloat16, __nv_bfloat16>, grid, PREP_WARPS * 32, smem, stream,
                   (const __nv_bfloat16*)u, u_stride, q_col, k_col, v_col, (const __nv_bfloat16*)q_norm_w,
-                  (const __nv_bfloat16*)k_norm_w, eps, inv_freq, rot_dims, halves, maps, mag, (__nv_bfloat16*)q_out, c, v_dim,
+                  (const __nv_bfloat16*)k_norm_w, unit_norm, eps, inv_freq, rot_dims, halves, maps, mag, (__nv_bfloat16*)q_out, c, v_dim,
                   positions, row_seq, q_heads, write_cache, bias, v_mix_in, v_mix, v_mix_out);
   else
     return ERR_BAD_DTYPE;

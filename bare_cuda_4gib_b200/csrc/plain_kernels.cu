@@ -704,6 +704,34 @@ static int glu_launch(const void* in, int in_dtype, int n_partials, long long pa
   return launch_status();
 }
 
+// ------------------------------------------------------------------------ cap on the logits
+
+// x <- cap * tanh(x / cap), element by element, four at a time where the length allows it.
+__global__ void softcap_rows_kernel(float* __restrict__ x, long long total, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float inv = 1.0f / cap;
+  const long long n4 = total / 4, at = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  float4* x4 = reinterpret_cast<float4*>(x);
+  for (long long i = at; i < n4; i += (long long)gridDim.x * blockDim.x) {
+    float4 v = x4[i];
+    v.x = cap * tanhf(v.x * inv); v.y = cap * tanhf(v.y * inv);
+    v.z = cap * tanhf(v.z * inv); v.w = cap * tanhf(v.w * inv);
+    x4[i] = v;
+  }
+  if (at < total - 4 * n4) x[4 * n4 + at] = cap * tanhf(x[4 * n4 + at] * inv);
+}
+
+extern "C" int llm_softcap_rows(float* logits, int rows, int vocab, float cap, cudaStream_t stream) {
+  const long long total = (long long)rows * vocab;
+  if (total <= 0) return 0;
+  LLM_HOST_CHECK(cap > 0.0f, ERR_BAD_SIZE);
+  LLM_HOST_CHECK(((uintptr_t)logits & 15) == 0, ERR_BAD_ALIGN);
+  const long long want = (total / 4 + 255) / 256;
+  launch_kernel(softcap_rows_kernel, (int)(want < 1 ? 1 : (want < 148 * 8 ? want : 148 * 8)), 256, 0, stream, logits, total, cap);
+  return launch_status();
+}
+
 // ------------------------------------------------------------------------------- sampling
 
 // One block per row: the index of the largest logit; the lowest index wins a tie.

@@ -1,8 +1,9 @@
 // Norms of a residual stream whose sublayers are normed on both sides:
 //
-//   x <- x + rms_norm(y) * b,   h = rms_norm(x) * w          (y a sublayer's result, h the next one's input)
+//   x <- x + m * rms_norm(y) * b,   h = rms_norm(x) * w      (y a sublayer's result, h the next one's input)
 //
-// as one kernel per sublayer boundary, and the embedding lookup followed by an RMS norm.  The
+// as one kernel per sublayer boundary (m a constant, 1 for most designs; without w, for sublayers that read
+// the stream un-normed, h = x), and the embedding lookup followed by an RMS norm.  The
 // stream, the sums of squares and both factors are float32; rms_norm(v) = v / sqrt(mean(v^2) + eps).
 // One block of a fixed size per row: the order of every sum depends on the width only.
 
@@ -55,12 +56,12 @@ extern "C" int llm_embed_rmsnorm(const void* table, const int32_t* ids, const vo
 }
 
 // One block per output row r (stream row src = row_index[r] or r).  With y: the partial results are
-// added in index order, normed with `post_w` and added into the stream, which is written back.
-// With out: the norm of the (new) stream row with `next_w`.
+// added in index order, normed with `post_w`, multiplied by `mult` and added into the stream, which is
+// written back.  With out: the norm of the (new) stream row with `next_w`, or without it the row itself.
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(NORM_THREADS)
 postnorm_add_rmsnorm_kernel(float* __restrict__ residual, const float* __restrict__ y, int n_partials,
-                            long long partial_stride, const TW* __restrict__ post_w, float post_eps,
+                            long long partial_stride, const TW* __restrict__ post_w, float post_eps, float mult,
                             const TW* __restrict__ next_w, float next_eps, TO* __restrict__ out,
                             const int32_t* __restrict__ row_index, int hidden) {
   pdl_launch_dependents();
@@ -78,7 +79,7 @@ postnorm_add_rmsnorm_kernel(float* __restrict__ residual, const float* __restric
       row_cache[i] = v;
       sq += v * v;
     }
-    const float s1 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + post_eps);
+    const float s1 = mult / sqrtf(block_sum(sq, scratch) / (float)hidden + post_eps);
     sq = 0.0f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
       const float v = x[i] + row_cache[i] * s1 * to_float(post_w[i]);
@@ -94,8 +95,12 @@ postnorm_add_rmsnorm_kernel(float* __restrict__ residual, const float* __restric
     }
   }
   if (!out) return;
-  const float s2 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + next_eps);
   TO* dst = out + (long long)r * hidden;
+  if (!next_w) {
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = from_float<TO>(row_cache[i]);
+    return;
+  }
+  const float s2 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + next_eps);
   for (int i = threadIdx.x; i < hidden; i += blockDim.x)
     dst[i] = from_float<TO>(row_cache[i] * s2 * to_float(next_w[i]));
 }
@@ -111,7 +116,7 @@ __device__ __forceinline__ float4 bf16x4(const __nv_bfloat16* p) {
 
 __global__ void __launch_bounds__(NORM_THREADS)
 postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __restrict__ y, int n_partials,
-                                long long partial_stride, const __nv_bfloat16* __restrict__ post_w, float post_eps,
+                                long long partial_stride, const __nv_bfloat16* __restrict__ post_w, float post_eps, float mult,
                                 const __nv_bfloat16* __restrict__ next_w, float next_eps, __nv_bfloat16* __restrict__ out,
                                 const int32_t* __restrict__ row_index, int hidden) {
   pdl_launch_dependents();
@@ -128,7 +133,7 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
     const int i = threadIdx.x + j * NORM_THREADS;
     if (i < n4) {
       old[j] = x[i];
-      float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      float4 a = y ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : old[j];
       for (int p = 0; p < n_partials; ++p) {
         const float4 d = reinterpret_cast<const float4*>(y + p * partial_stride + src * hidden)[i];
         a.x += d.x; a.y += d.y; a.z += d.z; a.w += d.w;
@@ -137,28 +142,30 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
       sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
     }
   }
-  const float s1 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + post_eps);
-  sq = 0.0f;
+  if (y) {
+    const float s1 = mult / sqrtf(block_sum(sq, scratch) / (float)hidden + post_eps);
+    sq = 0.0f;
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = threadIdx.x + j * NORM_THREADS;
-    if (i < n4) {
-      const float4 w = bf16x4(post_w + 4 * i);
-      float4 a = old[j];
-      a.x += v[j].x * s1 * w.x; a.y += v[j].y * s1 * w.y; a.z += v[j].z * s1 * w.z; a.w += v[j].w * s1 * w.w;
-      x[i] = a;
-      v[j] = a;
-      sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+    for (int j = 0; j < 4; ++j) {
+      const int i = threadIdx.x + j * NORM_THREADS;
+      if (i < n4) {
+        const float4 w = bf16x4(post_w + 4 * i);
+        float4 a = old[j];
+        a.x += v[j].x * s1 * w.x; a.y += v[j].y * s1 * w.y; a.z += v[j].z * s1 * w.z; a.w += v[j].w * s1 * w.w;
+        x[i] = a;
+        v[j] = a;
+        sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+      }
     }
   }
   if (!out) return;
-  const float s2 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + next_eps);
+  const float s2 = next_w ? 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + next_eps) : 1.0f;
   uint2* dst = reinterpret_cast<uint2*>(out + (long long)r * hidden);
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     const int i = threadIdx.x + j * NORM_THREADS;
     if (i < n4) {
-      const float4 w = bf16x4(next_w + 4 * i);
+      const float4 w = next_w ? bf16x4(next_w + 4 * i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
       const __nv_bfloat162 lo = __floats2bfloat162_rn(v[j].x * s2 * w.x, v[j].y * s2 * w.y);
       const __nv_bfloat162 hi = __floats2bfloat162_rn(v[j].z * s2 * w.z, v[j].w * s2 * w.w);
       uint2 o;
@@ -169,28 +176,30 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
   }
 }
 
-// dtype: the element type of the norm weights and of `out` (the step's activation type).
+// dtype: the element type of the norm weights and of `out` (the step's activation type).  y == nullptr: nothing
+// is added; next_w == nullptr: `out` gets the stream row itself.
 extern "C" int llm_postnorm_add_rmsnorm(float* residual, const float* y, int n_partials, long long partial_stride,
-                                        const void* post_w, float post_eps, const void* next_w, float next_eps,
+                                        const void* post_w, float post_eps, float mult, const void* next_w, float next_eps,
                                         void* out, int dtype, const int32_t* row_index, int rows, int hidden,
                                         cudaStream_t stream) {
   if (rows <= 0) return 0;
   const size_t smem = (size_t)(hidden + 32) * sizeof(float);
   LLM_HOST_CHECK(smem <= 48 * 1024, ERR_BAD_SIZE);
-  LLM_HOST_CHECK((!y || post_w) && (!out || next_w), ERR_BAD_SIZE);
+  LLM_HOST_CHECK(!y || post_w, ERR_BAD_SIZE);
+  if (!y) n_partials = 0;
   if (dtype == DT_F32)
     launch_kernel(postnorm_add_rmsnorm_kernel<float, float>, rows, NORM_THREADS, smem, stream, residual, y, n_partials,
-                  partial_stride, (const float*)post_w, post_eps, (const float*)next_w, next_eps, (float*)out, row_index,
+                  partial_stride, (const float*)post_w, post_eps, mult, (const float*)next_w, next_eps, (float*)out, row_index,
                   hidden);
-  else if (dtype == DT_BF16 && y && hidden % 4 == 0 && hidden <= 16 * NORM_THREADS && partial_stride % 4 == 0 &&
+  else if (dtype == DT_BF16 && hidden % 4 == 0 && hidden <= 16 * NORM_THREADS && partial_stride % 4 == 0 &&
            ((uintptr_t)residual % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)post_w % 8) == 0 &&
            ((uintptr_t)next_w % 8) == 0 && ((uintptr_t)out % 8) == 0)
     launch_kernel(postnorm_add_rmsnorm_vec_kernel, rows, NORM_THREADS, 0, stream, residual, y, n_partials, partial_stride,
-                  (const __nv_bfloat16*)post_w, post_eps, (const __nv_bfloat16*)next_w, next_eps, (__nv_bfloat16*)out,
+                  (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w, next_eps, (__nv_bfloat16*)out,
                   row_index, hidden);
   else if (dtype == DT_BF16)
     launch_kernel(postnorm_add_rmsnorm_kernel<__nv_bfloat16, __nv_bfloat16>, rows, NORM_THREADS, smem, stream, residual,
-                  y, n_partials, partial_stride, (const __nv_bfloat16*)post_w, post_eps, (const __nv_bfloat16*)next_w,
+                  y, n_partials, partial_stride, (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w,
                   next_eps, (__nv_bfloat16*)out, row_index, hidden);
   else
     return ERR_BAD_DTYPE;

@@ -17,7 +17,7 @@ import torch
 
 from . import build
 from ..errors import KernelLaunchError
-from .lib import CacheView, _check, sm_count
+from .lib import AttentionExtras, CacheView, _check, sm_count
 
 KEY_BLOCK = 64
 COUNTER_WORDS = 4096          # per-tile split counters at the start of the scratch (see the kernel)
@@ -53,7 +53,8 @@ def lib(head_dim: int, distance_bias: bool = False, v_dim: Optional[int] = None,
         l.llm_attention_mma.argtypes = [P, P, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, I, P, I, F, I, P]
         l.llm_attention_mma.restype = c_int
         if not distance_bias:
-            l.llm_attention_mma_general.argtypes = [P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, P, I, I, I, P, I, F, I, F, P]
+            l.llm_attention_mma_general.argtypes = [P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, P, I, I, I, P, I, F, I, F, I, P, P, L,
+                                                    P]
             l.llm_attention_mma_general.restype = c_int
         if distance_bias:
             l.llm_attention_mma_bias.argtypes = [P, P, L, F, P, I, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, I, P, I,
@@ -72,7 +73,7 @@ def tc_lib(head_dim: int):
     if l is None:
         l = build.load_library("attention_tcgen05.cu", defines(head_dim))
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
-        l.llm_attention_tcgen05.argtypes = [P, P, I, P, P, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, F, I, P, P]
+        l.llm_attention_tcgen05.argtypes = [P, P, I, P, P, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, F, I, I, P, P, L, P, P]
         l.llm_attention_tcgen05.restype = c_int
         l.llm_attention_tc_pool_map.argtypes = [P, P, L, I]
         l.llm_attention_tc_pool_map.restype = c_int
@@ -87,7 +88,8 @@ def decode_lib(head_dim: int):
     if l is None:
         l = build.load_library("attention_decode.cu", defines(head_dim))
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
-        l.llm_attention_decode.argtypes = [P, P, L, I, P, P, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, I, I, F, I, P, P]
+        l.llm_attention_decode.argtypes = [P, P, L, I, P, P, P, P, P, L, I, I, I, I, P, P, P, P, P, I, I, I, I, F, I, I, P, P, L,
+                                           P, P]
         l.llm_attention_decode.restype = c_int
         l.llm_attention_decode_pool_map.argtypes = [P, P, L, I]
         l.llm_attention_decode_pool_map.restype = c_int
@@ -99,15 +101,17 @@ def decode_lib(head_dim: int):
 
 class AttentionPlan:
     def __init__(self, head_dim: int, heads: int, kv_heads: int, distance_bias: bool = False,
-                 v_dim: Optional[int] = None, softcap: float = 0.0):
+                 v_dim: Optional[int] = None, softcap: float = 0.0, span: Optional[int] = None):
         """`distance_bias`: attention whose scores get a bias by distance; `v_dim`: value heads of a size of
         their own; `softcap` > 0: scaled scores capped with a tanh.  Only the mma.sync kernel has these
-        variants, so such a plan uses it for every step shape."""
+        variants, so such a plan uses it for every step shape.  `span` (None: no bound): how many keys a query
+        sees at most, which bounds how often a decode step's keys are worth splitting."""
         self.head_dim, self.heads, self.kv_heads = head_dim, heads, kv_heads
         self.group = heads // kv_heads
         self.distance_bias = distance_bias
         self.v_dim = head_dim if v_dim is None else int(v_dim)
         self.softcap = float(softcap or 0.0)
+        self.span = int(span) if span else None
         self.general = self.v_dim != head_dim or self.softcap > 0.0      # what only the mma.sync kernel computes
         self.lib = lib(head_dim, distance_bias, self.v_dim, self.softcap > 0.0)
         self.prefill_rows = int(self.lib.llm_attention_prefill_rows())
@@ -187,16 +191,16 @@ class AttentionPlan:
 
 
 def plan_for(head_dim: int, heads: int, kv_heads: int, distance_bias: bool = False, v_dim: Optional[int] = None,
-             softcap: float = 0.0) -> Optional[AttentionPlan]:
+             softcap: float = 0.0, span: Optional[int] = None) -> Optional[AttentionPlan]:
     if not supports(head_dim, v_dim) or (distance_bias and (softcap or (v_dim or head_dim) != head_dim)):
         return None
-    return AttentionPlan(head_dim, heads, kv_heads, distance_bias, v_dim, softcap)
+    return AttentionPlan(head_dim, heads, kv_heads, distance_bias, v_dim, softcap, span)
 
 
 def step_tiles(ctx, plan: AttentionPlan):
     """The step's row tiles for this head grouping: built once per step and shared by all layers."""
     key = ("attention_tiles", plan.group, plan.kv_heads, plan.head_dim, plan.distance_bias, plan.prefill_rows,
-           plan.decode is not None)
+           plan.decode is not None, plan.span)
     cached = ctx.extras.get(key)
     if cached is not None:
         return cached
@@ -220,6 +224,8 @@ def step_tiles(ctx, plan: AttentionPlan):
     use_decode = rows_per_tile == 16 and plan.decode is not None and n_tiles * plan.kv_heads <= DECODE_MAX_TILES
     if rows_per_tile == 16 and not use_decode:
         key_blocks = -(-ctx.max_kv_len // KEY_BLOCK)
+        if plan.span:      # a tile's rows see `span` keys each, at most max_q_len positions apart
+            key_blocks = min(key_blocks, -(-(plan.span + ctx.max_q_len) // KEY_BLOCK) + 1)
         n_splits = max(1, min(key_blocks, -(-(2 * sm_count()) // (n_tiles * plan.kv_heads))))
         if os.environ.get("BARE_CUDA_B200_ATTN_SPLITS"):     # experiments only
             n_splits = min(key_blocks, int(os.environ["BARE_CUDA_B200_ATTN_SPLITS"]))
@@ -252,9 +258,14 @@ def usable_with_bias(out: torch.Tensor, cache: CacheView) -> bool:
 
 
 def run(ctx, plan: AttentionPlan, q: torch.Tensor, out: torch.Tensor, cache: CacheView, scale: float,
-        window: int, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+        window: int, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+        extras: Optional[AttentionExtras] = None) -> None:
     """`bias` (float32 [heads, distances], plans made with `distance_bias` only) is added to the
-    scaled scores by distance; such a plan may write a column view and scales its output."""
+    scaled scores by distance; such a plan may write a column view and scales its output.  `extras`
+    (other plans): blocks of positions, sink, gate."""
+    more = (extras or AttentionExtras()).arguments(plan.heads, q.dtype)
+    if plan.distance_bias and extras:
+        raise KernelLaunchError("attention_mma (distance bias): the variant takes no blocks of positions, sink or gate")
     tile_seq, tile_index, n_tiles, rows_per_tile, n_splits, dec_splits, dec_slots = step_tiles(ctx, plan)
     if plan.distance_bias:
         scratch_ptr = 0
@@ -276,7 +287,7 @@ def run(ctx, plan: AttentionPlan, q: torch.Tensor, out: torch.Tensor, cache: Cac
             out.data_ptr(), cache.k_ptr, cache.v_ptr, cache.block_table.data_ptr(), cache.page_stride,
             cache.table_stride, cache.page_tokens, cache.kv_heads, cache.head_dim, ctx.seq_q_start.data_ptr(),
             ctx.seq_q_len.data_ptr(), ctx.seq_kv_len.data_ptr(), tile_seq.data_ptr(), tile_index.data_ptr(), n_tiles,
-            dec_splits, dec_slots, plan.heads, scale, window, gemm.error_word(q.device).data_ptr(), ctx.stream),
+            dec_splits, dec_slots, plan.heads, scale, window, *more, gemm.error_word(q.device).data_ptr(), ctx.stream),
             "attention_decode")
         return
     if plan.tc is not None and rows_per_tile != 16:
@@ -289,21 +300,21 @@ def run(ctx, plan: AttentionPlan, q: torch.Tensor, out: torch.Tensor, cache: Cac
             ctypes.addressof(pool_map), cache.pool_ptr, box_rows, q.data_ptr(), out.data_ptr(), cache.k_ptr, cache.v_ptr, cache.block_table.data_ptr(), cache.page_stride,
             cache.table_stride, cache.page_tokens, cache.kv_heads, cache.head_dim, ctx.seq_q_start.data_ptr(),
             ctx.seq_q_len.data_ptr(), ctx.seq_kv_len.data_ptr(), tile_seq.data_ptr(), tile_index.data_ptr(), n_tiles,
-            plan.heads, scale, window, gemm.error_word(q.device).data_ptr(), ctx.stream), "attention_tcgen05")
+            plan.heads, scale, window, *more, gemm.error_word(q.device).data_ptr(), ctx.stream), "attention_tcgen05")
         return
     scratch_ptr = 0
     if n_splits > 1:
         floats = plan.lib.llm_attention_scratch_floats(n_tiles, plan.kv_heads, n_splits, rows_per_tile)
         scratch_ptr = plan.scratch(ctx, int(floats), q.device).data_ptr()
-    if plan.general:
+    if plan.general or extras:
         if cache.v_dim != plan.v_dim or cache.head_dim != plan.head_dim:
             raise KernelLaunchError("attention_mma: the cache's head sizes are not the plan's")
         _check(plan.lib.llm_attention_mma_general(
             q.data_ptr(), out.data_ptr(), cache.k_ptr, cache.v_ptr, cache.block_table.data_ptr(), cache.page_stride,
             cache.table_stride, cache.page_tokens, cache.kv_heads, cache.head_dim, cache.v_dim, ctx.seq_q_start.data_ptr(),
             ctx.seq_q_len.data_ptr(), ctx.seq_kv_len.data_ptr(), tile_seq.data_ptr(), tile_index.data_ptr(), n_tiles,
-            rows_per_tile, n_splits, scratch_ptr, plan.heads, scale, window, plan.softcap, ctx.stream),
-            "attention_mma (value size, score cap)")
+            rows_per_tile, n_splits, scratch_ptr, plan.heads, scale, window, plan.softcap, *more, ctx.stream),
+            "attention_mma (value size, score cap, extras)")
         return
     _check(plan.lib.llm_attention_mma(
         q.data_ptr(), out.data_ptr(), cache.k_ptr, cache.v_ptr, cache.block_table.data_ptr(), cache.page_stride,

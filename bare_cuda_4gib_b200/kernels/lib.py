@@ -88,6 +88,30 @@ class CacheView:
         self.dtype = dtype
 
 
+class AttentionExtras:
+    """What a softmax-attention kernel may be given beside its queries and its cache: `chunk` (0: none;
+    a query sees its own block of that many positions only, blocks counted from position 0), `sink`
+    (float32 [heads]: exp(sink) joins each head's denominator once), `gate` (a [rows, heads] column view
+    in the step's element type: head h's output is multiplied by sigmoid(gate[row, h]))."""
+
+    __slots__ = ("chunk", "sink", "gate")
+
+    def __init__(self, chunk: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
+        self.chunk, self.sink, self.gate = int(chunk), sink, gate
+
+    def arguments(self, heads: int, dtype: torch.dtype):
+        """The last arguments of the kernels' entry points: chunk, sink, gate, gate row stride."""
+        _dev(self.sink, self.gate)
+        if self.sink is not None and (self.sink.dtype != torch.float32 or self.sink.numel() != heads or not self.sink.is_contiguous()):
+            raise KernelLaunchError(f"attention: the sink must be float32 with one number for each of the {heads} heads")
+        if self.gate is not None and (self.gate.dtype != dtype or self.gate.shape[-1] != heads or self.gate.stride(-1) != 1):
+            raise KernelLaunchError(f"attention: the gate must have the step's element type and one column for each of the {heads} heads")
+        return self.chunk, _ptr(self.sink), _ptr(self.gate), self.gate.stride(0) if self.gate is not None else 0
+
+    def __bool__(self) -> bool:
+        return bool(self.chunk) or self.sink is not None or self.gate is not None
+
+
 class _Plain:
     def __init__(self):
         lib = build.load_library("plain_kernels.cu")
@@ -100,10 +124,12 @@ class _Plain:
         lib.llm_swiglu.argtypes = [P, I, I, L, P, I, I, I, P]
         lib.llm_glu.argtypes = [P, I, I, L, P, I, I, I, I, P]
         lib.llm_glu_clamped.argtypes = [P, I, I, L, P, I, I, I, F, F, P]
+        lib.llm_softcap_rows.argtypes = [P, I, I, F, P]
         lib.llm_argmax_rows.argtypes = [P, P, I, I, P]
         lib.llm_sample_rows.argtypes = [P, P, P, P, I, I, P]
         for name in ("llm_embed_gather", "llm_add_rmsnorm", "llm_matmul_plain", "llm_rope_cache_write",
-                     "llm_attention_plain", "llm_swiglu", "llm_glu", "llm_glu_clamped", "llm_argmax_rows", "llm_sample_rows"):
+                     "llm_attention_plain", "llm_swiglu", "llm_glu", "llm_glu_clamped", "llm_softcap_rows",
+                     "llm_argmax_rows", "llm_sample_rows"):
             getattr(lib, name).restype = c_int
         self.lib = lib
 
@@ -315,6 +341,15 @@ def glu_clamped(gate_up: Partials, out: torch.Tensor, n_tokens: int, limit: floa
                                        gate_up.stride, out.data_ptr(), dtype_code(out.dtype), n_tokens, out.shape[-1],
                                        float(limit), float(alpha), stream if stream is not None else stream_handle()),
            "glu_clamped")
+
+
+def softcap_rows(logits: torch.Tensor, cap: float, rows: int, stream=None) -> None:
+    """logits[:rows] = cap * tanh(logits / cap), float32, in place."""
+    _dev(logits)
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise TypeError("softcap_rows: the logits must be contiguous float32")
+    _check(plain().lib.llm_softcap_rows(logits.data_ptr(), rows, logits.shape[-1], float(cap),
+                                        stream if stream is not None else stream_handle()), "softcap_rows")
 
 
 def argmax_rows(logits: torch.Tensor, out: torch.Tensor, rows: int, stream=None) -> None:

@@ -213,16 +213,23 @@ class GeneralAttention(Part):
     `rotary_pairs`, `none`); a `scale` of its own; a cap on the scaled scores, cap * tanh(score / cap);
     value heads of their own size; a `window`; and value mixing: with `v_mix` = "source" the values this
     layer caches are also left for later layers of the step, with "mix" the cached value is (1 - l) v +
-    l v_source of the same token, l the scalar tensor `v_lambda`.
+    l v_source of the same token, l the scalar tensor `v_lambda`; queries and keys divided by their root
+    mean square per head after the rotation (`unit_qk`, without weights); blocks of positions (`chunk`: a
+    query sees its own block only, blocks counted from position 0); a learned number per head whose
+    exponential joins the softmax's denominator (`sink`); and one sigmoid gate per head on its output,
+    read from the mixer's input (`head_gate`).
 
-    One product makes [q | k | v]; one kernel adds the biases, norms, turns, mixes and caches; then the
+    One product makes [q | k | v (| g)]; one kernel adds the biases, norms, turns, mixes and caches; then the
     engine's tensor-core attention kernels run in bfloat16 steps (all three for equal key and value sizes
     without a cap, the mma.sync kernel built for the value size and the cap otherwise), the plain kernel in
-    float32 steps and for sizes that are no multiples of 16 up to 128.
+    float32 steps and for sizes that are no multiples of 16 up to 128.  All of them join the sink and apply
+    the gate where they finish a row.
 
     params: `hidden`, `heads`, `kv_heads`, `dim`, `vdim`, `scale`, `eps`, `bias` (bool), `qk_norm` (bool),
-    `softcap` (None: no cap), `window` (None: every key), `v_mix` (None | "source" | "mix"), `position`.
-    tensors: `q`, `k`, `v`, `o`, (`q_bias`, `k_bias`, `v_bias`,) (`q_norm`, `k_norm` [dim],) (`v_lambda` [])."""
+    `unit_qk` (bool), `softcap` (None: no cap), `window`, `chunk` (None: every key), `sink` (bool), `head_gate`
+    (bool), `v_mix` (None | "source" | "mix"), `position`.
+    tensors: `q`, `k`, `v`, `o`, (`q_bias`, `k_bias`, `v_bias`,) (`q_norm`, `k_norm` [dim],) (`v_lambda` [],)
+    (`sink` [heads],) (`g` [heads, hidden])."""
 
     takes_lazy_input = False
 
@@ -236,7 +243,11 @@ class GeneralAttention(Part):
         if self.vdim > 256:
             raise ConfigError(f"general_attention: value head size {self.vdim} exceeds the 256 the kernels take")
         self.window = p.get("window")
-        self.has_bias, self.qk_norm = bool(p.get("bias")), bool(p.get("qk_norm"))
+        self.chunk = p.get("chunk")
+        self.has_bias, self.qk_norm, self.unit_qk = bool(p.get("bias")), bool(p.get("qk_norm")), bool(p.get("unit_qk"))
+        if self.qk_norm and self.unit_qk:
+            raise ConfigError("general_attention: queries and keys are normed with weights or without, not both")
+        self.has_sink, self.head_gate = bool(p.get("sink")), bool(p.get("head_gate"))
         self.softcap = float(p["softcap"]) if p.get("softcap") else 0.0
         self.v_mix = p.get("v_mix")
         if self.v_mix not in (None, "source", "mix"):
@@ -258,20 +269,32 @@ class GeneralAttention(Part):
             out.update({"q_norm": ((self.dim,), "norm"), "k_norm": ((self.dim,), "norm")})
         if self.v_mix is not None:
             out["v_lambda"] = ((), "zero")      # the source layer has the tensor too and does not use it
+        if self.has_sink:
+            out["sink"] = ((self.heads,), "unit")
+        if self.head_gate:
+            out["g"] = ((self.heads, self.hidden), "matrix")
         return out
 
+    def _projections(self):
+        return ("q", "k", "v", "g") if self.head_gate else ("q", "k", "v")
+
     def adjacent_weights(self):
-        return [("q", "k", "v")]
+        return [self._projections()]
+
+    def _span(self):
+        """How many keys a query sees at most: its window, and never more than one block of `chunk` positions."""
+        spans = [int(s) for s in (self.window, self.chunk) if s]
+        return min(spans) if spans else None
 
     def cache_request(self):
-        return KVCacheRequest(self.kv_heads, self.dim, self.window, None if self.vdim == self.dim else self.vdim)
+        return KVCacheRequest(self.kv_heads, self.dim, self._span(), None if self.vdim == self.dim else self.vdim)
 
     def state_request(self):
         return None
 
     def prepare(self, dtype, device) -> None:
         t = self.tensors
-        self.proj = Linear(fused_rows([t["q"], t["k"], t["v"]]), "general_attention.in")
+        self.proj = Linear(fused_rows([t[n] for n in self._projections()]), "general_attention.in")
         self.o = Linear(t["o"], "general_attention.o")
         self.proj.prepare(dtype)
         self.o.prepare(dtype)
@@ -287,12 +310,15 @@ class GeneralAttention(Part):
             raise ConfigError(f"general_attention: {self.rot_dims} rotated entries in a head of {self.dim}")
         self.halves = bool(getattr(self.position, "halves", False))
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
+        if self.unit_qk and self.magnitude != 1.0:
+            raise ConfigError("general_attention: queries and keys of unit size take a rotation that keeps their size")
+        self.sink = t["sink"].to(torch.float32).contiguous() if self.has_sink else None
         self.fast = None
         if dtype == torch.bfloat16 and device.type == "cuda":
             # equal head sizes without a cap: the engine's tcgen05 prefill, cluster decode and mma.sync kernels;
             # otherwise the mma.sync kernel built for this value size and with the cap (sizes it takes)
             from ..kernels import attention as fast
-            self.fast = fast.plan_for(self.dim, self.heads, self.kv_heads, False, self.vdim, self.softcap)
+            self.fast = fast.plan_for(self.dim, self.heads, self.kv_heads, False, self.vdim, self.softcap, self._span())
 
     def plan_step(self, ctx) -> None:
         if self.fast is not None and ctx.use_fast_attention:
@@ -308,12 +334,14 @@ class GeneralAttention(Part):
         HP.headnorm_rope_cache(ctx, u, 0, self.qd, self.qd + self.kd, self.q_norm, self.k_norm, self.eps, self.inv_freq,
                                self.rot_dims, self.magnitude, q, call.cache, self.heads, call.writes_cache,
                                halves=self.halves, bias=self.bias, v_mix_in=shared if self.v_mix == "mix" else None,
-                               v_mix=self.v_lambda, v_mix_out=shared if self.v_mix == "source" else None)
+                               v_mix=self.v_lambda, v_mix_out=shared if self.v_mix == "source" else None,
+                               unit_norm=self.unit_qk)
         out = ctx.ws.get("attn_out", (n, self.heads * self.vdim), ctx.dtype)
         window = int(self.window) if self.window else 0
+        extras = K.AttentionExtras(self.chunk or 0, self.sink, u[:, u.shape[1] - self.heads:] if self.head_gate else None)
         if self.fast is not None and ctx.use_fast_attention:
             from ..kernels import attention as fast
-            fast.run(ctx, self.fast, q, out, call.cache, self.scale, window)
+            fast.run(ctx, self.fast, q, out, call.cache, self.scale, window, extras=extras)
         else:
-            BA.attention(ctx, q, out, call.cache, None, self.heads, self.scale, window, 1.0, self.softcap)
+            BA.attention(ctx, q, out, call.cache, None, self.heads, self.scale, window, 1.0, self.softcap, extras)
         return self.o.forward(ctx, out, n, torch.float32, "attn_proj", allow_partials=True)

@@ -31,7 +31,8 @@ class TokenEmbedding(Part):
 
 @register_head("linear")
 class OutputHead(Part):
-    """params: `vocab`, `hidden`.  tensors: `weight` [vocab, hidden] (may be the embedding's)."""
+    """params: `vocab`, `hidden`, `softcap` (optional: every logit z becomes cap * tanh(z / cap)).
+    tensors: `weight` [vocab, hidden] (may be the embedding's)."""
 
     def local_weights(self):
         return {"weight": ((int(self.params["vocab"]), int(self.params["hidden"])), "matrix")}
@@ -43,7 +44,10 @@ class OutputHead(Part):
     takes_lazy_input = True
 
     def forward(self, ctx, normed, rows: int) -> torch.Tensor:
-        return self.linear.forward(ctx, normed, rows, torch.float32, "logits").tensor
+        logits = self.linear.forward(ctx, normed, rows, torch.float32, "logits").tensor
+        if self.params.get("softcap"):
+            K.softcap_rows(logits, float(self.params["softcap"]), rows, ctx.stream)
+        return logits
 
 
 @register_embedding("table_positions")

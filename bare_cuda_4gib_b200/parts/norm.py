@@ -63,9 +63,10 @@ class SandwichRMSNorm(Part):
     """RMS norm of a stream whose sublayers are normed on both sides, x <- x + norm_b(f(norm(x))).
     As the norm before a sublayer it first adds what is pending, a `NormedDelta` (the previous
     sublayer's result with the weight of its norm behind), in the same kernel; as the norm behind a
-    sublayer it only lends its weight (`pending`).
+    sublayer it only lends its weight (`pending`).  With `mult` the normed result is multiplied by that
+    constant before it is added.
 
-    params: `size`, `eps`.  tensors: `weight` [size]."""
+    params: `size`, `eps`, `mult` (optional, of the norm behind).  tensors: `weight` [size]."""
 
     def local_weights(self):
         return {"weight": ((self.params["size"],), "norm")}
@@ -75,13 +76,29 @@ class SandwichRMSNorm(Part):
 
     def pending(self, y):
         from ..kernels.sandwich import NormedDelta
-        return NormedDelta(y, self.weight, float(self.params["eps"]))
+        return NormedDelta(y, self.weight, float(self.params["eps"]), float(self.params.get("mult", 1.0)))
 
     def forward(self, ctx, residual: torch.Tensor, delta, rows: int, row_index: Optional[torch.Tensor] = None,
                 buffer: str = "normed", lazy: bool = False):
         from ..kernels import sandwich as SW
         out = ctx.ws.get(buffer, (rows, self.params["size"]), ctx.dtype)
         SW.postnorm_add_rmsnorm(residual, delta, self.weight, out, float(self.params["eps"]), rows, row_index, ctx.stream)
+        return out
+
+
+@register_norm("stream_input")
+class StreamInput(Part):
+    """What stands ahead of a sublayer that reads the residual stream itself: it carries out what is
+    pending (a `NormedDelta`, as `SandwichRMSNorm` does) and hands the stream on in the step's
+    activation type, un-normed, in the same kernel.
+
+    params: `size`.  No tensors."""
+
+    def forward(self, ctx, residual: torch.Tensor, delta, rows: int, row_index: Optional[torch.Tensor] = None,
+                buffer: str = "normed", lazy: bool = False):
+        from ..kernels import sandwich as SW
+        out = ctx.ws.get(buffer, (rows, self.params["size"]), ctx.dtype)
+        SW.postnorm_add_rmsnorm(residual, delta, None, out, 0.0, rows, row_index, ctx.stream)
         return out
 
 
