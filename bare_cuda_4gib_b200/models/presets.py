@@ -130,6 +130,29 @@ PRESETS.update({
 })
 
 
+def _fuzazen(width, vocab, ff, heads, kv_heads, dim, vdim, chunk, rot_dims, own, repeats):
+    """`own` layers with tensors of their own, all run `repeats` more times in the same order."""
+    layer = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+             "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk},
+                       "rot": {"base": 10000.0, "dims": rot_dims}, "scale": dim ** -0.5}}
+    layers = [layer] * own
+    for _ in range(repeats):
+        layers = layers + [dict(layer, weights_of=j) for j in range(own)]
+    return dict(architecture="Fuzazen", vocab=vocab, width=width, embedding={"scale": 1.0}, norm={"eps": 1e-6},
+                residual_mult=0.5, logit_softcap=30.0, layers=layers)
+
+
+PRESETS.update({
+    "fuzazen-tiny": _fuzazen(64, 300, 96, 4, 2, 16, 24, 20, 8, 2, 1),
+    # layer sizes of TinyLlama (width 2048, feed-forward 5632, 32 heads of 64, 4 key heads), blocks of 1,024 positions
+    "fuzazen-2048": _fuzazen(2048, 32000, 5632, 32, 4, 64, 64, 1024, 64, 4, 1),
+    # ... and of Llama-2-7B (width 4096, feed-forward 11008, 32 heads of 128)
+    "fuzazen-4096": _fuzazen(4096, 32000, 11008, 32, 32, 128, 128, 1024, 128, 4, 1),
+    # value heads of another size than the key heads', as the Gurolix presets have them
+    "fuzazen-2048-values": _fuzazen(2048, 32000, 5632, 16, 4, 128, 64, 1024, 64, 4, 1),
+})
+
+
 def preset_config(name: str, **overrides):
     from ..config.llama import LlamaConfig
     from ..errors import ConfigError
