@@ -304,6 +304,15 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
     const uint32_t k_base = smem_u32(my_kv) + slot * KV_BYTES, v_base = k_base + SUBS * SUB_BYTES;
     const int kb = kb_lo + gw + j * stride;
     const int key0 = kb * BN;
+    if (key0 + BN > kv_len) {
+      // the request's last key block: a page may hold anything behind the last key, and a weight of zero
+      // times NaN is not zero, so those value rows are cleared (no later block of this warp uses the slot)
+      for (int i = lane; i < (key0 + BN - kv_len) * SUBS * 8; i += 32) {
+        const int r = kv_len - key0 + i / (SUBS * 8), c = i % (SUBS * 8);
+        asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(v_base + (c / 8) * SUB_BYTES + r * 128 + (c % 8) * 16), "r"(0) : "memory");
+      }
+      __syncwarp();
+    }
 
     float s[NT][4];
 #pragma unroll

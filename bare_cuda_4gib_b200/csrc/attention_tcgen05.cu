@@ -438,7 +438,14 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
         for (int g = 0; g < TILES; ++g) any = any || pv_next[g] < n_g[g];
         return any;
       };
-      auto landed = [&](int n) { return mbar_try_wait(&tile_full[n % SLOTS], (n / SLOTS) & 1); };
+      // Whether tile n has landed.  A barrier's parity tells one filling of a slot only from the one before it, so
+      // the tiles are counted off in order: a group whose first key block lies several blocks behind the
+      // other's (it begins in a later block of positions) would else take an earlier filling for its own.
+      int arrived = 0;
+      auto landed = [&](int n) {
+        while (arrived <= n && mbar_try_wait(&tile_full[arrived % SLOTS], (arrived / SLOTS) & 1)) ++arrived;
+        return arrived > n;
+      };
       unsigned long long idle_since = 0;
       unsigned idle_spins = 0;
       while (ok && unfinished()) {

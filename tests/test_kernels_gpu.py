@@ -21,7 +21,7 @@ def _ctx(max_rows=4096):
 
 def _close(got, want, rtol, atol):
     got, want = got.double().cpu(), want.double().cpu()
-    bad = (got - want).abs() > atol + rtol * want.abs()
+    bad = ~((got - want).abs() <= atol + rtol * want.abs())        # NaN is bad too
     assert not bad.any(), f"{int(bad.sum())} of {bad.numel()} differ; worst {float((got - want).abs().max()):.3e}"
 
 
