@@ -100,6 +100,90 @@ headnorm_rope_cache_kernel(const T* __restrict__ u, long long u_stride, int q_co
   }
 }
 
+// The same with 16-byte accesses: bfloat16, neighbouring pairs, no bias and no value mixing, heads of 8, 16, 32,
+// 64, 128 or 256 entries.  A thread holds eight entries of a head (four pairs), so `d / 8` neighbouring lanes
+// of a warp hold a head and sum its squares among themselves; cos and sin are formed once per block and
+// pair instead of once per head.  Grid (token, share of the token's pieces).
+__global__ void __launch_bounds__(PREP_WARPS * 32)
+headnorm_rope_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, int q_col, int k_col, int v_col,
+                               const __nv_bfloat16* __restrict__ q_norm_w, const __nv_bfloat16* __restrict__ k_norm_w,
+                               int unit_norm, float eps, const float* __restrict__ inv_freq, int rot_dims, float mag,
+                               __nv_bfloat16* __restrict__ q_out, PagedCache cache, int v_dim,
+                               const int32_t* __restrict__ positions, const int32_t* __restrict__ row_seq, int q_heads,
+                               int write_cache) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float2 turn[128];       // cos and sin of the token's angles, times mag
+  const int t = blockIdx.x, d = cache.head_dim, lanes = d / 8;
+  const int pos = positions[t], seq = row_seq[t];
+  for (int p = threadIdx.x; p < rot_dims / 2; p += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * inv_freq[p], &sn, &cs);
+    turn[p] = make_float2(cs * mag, sn * mag);
+  }
+  __syncthreads();
+  const int page = write_cache ? cache.block_table[(long long)seq * cache.table_stride + pos / cache.page_tokens] : -1;
+  const long long in_page = pos % cache.page_tokens;
+  const __nv_bfloat16* row = u + (long long)t * u_stride;
+  const int turned = (q_heads + cache.kv_heads) * lanes;                       // pieces of q and k, then those of v
+  const int pieces = turned + (page >= 0 ? cache.kv_heads * (v_dim / 8) : 0);
+  // whole warps walk on together: a head's lanes lie in one warp and meet in its shuffles
+  for (int base = (blockIdx.y * blockDim.x + threadIdx.x) & ~31; base < pieces; base += gridDim.y * blockDim.x) {
+    const int w = base + (threadIdx.x & 31);
+    const bool is_qk = w < turned;
+    const int head = is_qk ? w / lanes : 0, part = is_qk ? w - head * lanes : 0;
+    const bool is_q = head < q_heads;
+    float x[8];
+    float sq = 0.0f;
+    if (is_qk) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(row + (is_q ? q_col + head * d : k_col + (head - q_heads) * d) + part * 8);
+      const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[j] = __bfloat162float(e[j]);
+        sq += x[j] * x[j];
+      }
+    }
+    for (int o = lanes / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if (is_qk) {
+      const __nv_bfloat16* nw = is_q ? q_norm_w : k_norm_w;
+      const float scale = nw || unit_norm ? 1.0f / sqrtf(sq / (float)d + eps) : 1.0f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] *= scale;
+      if (nw) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(nw + part * 8);
+        const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] *= __bfloat162float(e[j]);
+      }
+      uint4 packed;
+      __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float a = x[2 * j], b = x[2 * j + 1];
+        if (part * 8 + 2 * j < rot_dims) {
+          const float2 cs = turn[part * 4 + j];
+          const float na = a * cs.x - b * cs.y;
+          b = b * cs.x + a * cs.y;
+          a = na;
+        }
+        o2[j] = __floats2bfloat162_rn(a, b);
+      }
+      __nv_bfloat16* dst = nullptr;
+      if (is_q)
+        dst = q_out + ((long long)t * q_heads + head) * d;
+      else if (page >= 0)
+        dst = (__nv_bfloat16*)cache.k + (long long)page * cache.page_stride + ((long long)(head - q_heads) * cache.page_tokens + in_page) * d;
+      if (dst) *reinterpret_cast<uint4*>(dst + part * 8) = packed;
+    } else if (w < pieces) {
+      const int v = w - turned, g = v / (v_dim / 8), c = (v - g * (v_dim / 8)) * 8;
+      *reinterpret_cast<uint4*>((__nv_bfloat16*)cache.v + (long long)page * cache.page_stride +
+                                ((long long)g * cache.page_tokens + in_page) * v_dim + c) =
+          *reinterpret_cast<const uint4*>(row + (v_col >= 0 ? v_col : k_col) + g * v_dim + c);
+    }
+  }
+}
+
 // dtype: element type of u, q_out, the cache and the norm weights.
 extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_stride, int q_col, int k_col, int v_col,
                                        const void* q_norm_w, const void* k_norm_w, int unit_norm, float eps,
@@ -119,6 +203,20 @@ extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_str
   const size_t smem = (size_t)PREP_WARPS * head_dim * sizeof(float);
   LLM_HOST_CHECK(smem <= 48 * 1024, ERR_BAD_SIZE);
   PagedCache c{k_base, v_base, block_table, page_stride, table_stride, page_tokens, kv_heads, head_dim};
+  const auto whole = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool heads_fit = head_dim == 8 || head_dim == 16 || head_dim == 32 || head_dim == 64 || head_dim == 128 || head_dim == 256;
+  if (dtype == DT_BF16 && heads_fit && !halves && maps == 1 && !bias && !v_mix_in && !v_mix_out && v_dim % 8 == 0 &&
+      u_stride % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && (v_col < 0 || v_col % 8 == 0) && page_stride % 8 == 0 &&
+      whole(u) && whole(q_out) && whole(k_base) && whole(v_base) && whole(q_norm_w) && whole(k_norm_w)) {
+    const int pieces = (q_heads + kv_heads) * (head_dim / 8) + kv_heads * (v_dim / 8);
+    // few tokens: a token's pieces are dealt to several blocks
+    const int shares = n_tokens >= 256 ? 1 : (pieces + PREP_WARPS * 32 - 1) / (PREP_WARPS * 32);
+    launch_kernel(headnorm_rope_cache_vec_kernel, dim3(n_tokens, shares < 16 ? shares : 16), PREP_WARPS * 32, 0, stream,
+                  (const __nv_bfloat16*)u, u_stride, q_col, k_col, v_col, (const __nv_bfloat16*)q_norm_w,
+                  (const __nv_bfloat16*)k_norm_w, unit_norm, eps, inv_freq, rot_dims, mag, (__nv_bfloat16*)q_out, c, v_dim,
+                  positions, row_seq, q_heads, write_cache);
+    return launch_status();
+  }
   // few tokens: a token's heads are dealt to several blocks, so that the step still fills the GPU
   const int per_token = n_tokens >= 256 ? 1 : min(((q_heads + kv_heads) * maps + PREP_WARPS - 1) / PREP_WARPS, 16);
   const dim3 grid(n_tokens, per_token);

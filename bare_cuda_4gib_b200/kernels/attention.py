@@ -101,17 +101,19 @@ def decode_lib(head_dim: int):
 
 class AttentionPlan:
     def __init__(self, head_dim: int, heads: int, kv_heads: int, distance_bias: bool = False,
-                 v_dim: Optional[int] = None, softcap: float = 0.0, span: Optional[int] = None):
+                 v_dim: Optional[int] = None, softcap: float = 0.0, window: Optional[int] = None,
+                 chunk: Optional[int] = None):
         """`distance_bias`: attention whose scores get a bias by distance; `v_dim`: value heads of a size of
         their own; `softcap` > 0: scaled scores capped with a tanh.  Only the mma.sync kernel has these
-        variants, so such a plan uses it for every step shape.  `span` (None: no bound): how many keys a query
-        sees at most, which bounds how often a decode step's keys are worth splitting."""
+        variants, so such a plan uses it for every step shape.  `window` and `chunk` (None: no bound): what the
+        calls will say; here they bound how often a decode step's keys are worth splitting, and `chunk` orders
+        a prompt's tiles by the keys they see."""
         self.head_dim, self.heads, self.kv_heads = head_dim, heads, kv_heads
         self.group = heads // kv_heads
         self.distance_bias = distance_bias
         self.v_dim = head_dim if v_dim is None else int(v_dim)
         self.softcap = float(softcap or 0.0)
-        self.span = int(span) if span else None
+        self.window, self.chunk = int(window or 0), int(chunk or 0)
         self.general = self.v_dim != head_dim or self.softcap > 0.0      # what only the mma.sync kernel computes
         self.lib = lib(head_dim, distance_bias, self.v_dim, self.softcap > 0.0)
         self.prefill_rows = int(self.lib.llm_attention_prefill_rows())
@@ -128,6 +130,16 @@ class AttentionPlan:
         self._scratch = None
         self._pool_maps = {}
         self._decode_maps = {}
+
+    def key_blocks(self, kv_len: int, q_len: int, block: int) -> int:
+        """The most blocks of `block` keys that one tile of a request reads: `kv_len` keys, `q_len` tokens."""
+        n = -(-kv_len // block)
+        if self.window:
+            n = min(n, -(-(self.window + q_len - 2) // block) + 1)
+        if self.chunk:
+            whole = q_len == 1 and self.chunk % block == 0      # blocks of positions that begin with a block of keys
+            n = min(n, self.chunk // block if whole else -(-(self.chunk + q_len - 2) // block) + 1)
+        return n
 
     def decode_map(self, cache: CacheView):
         """The decode kernel's tensor map over a cache group's pool (boxes of at most 64 rows)."""
@@ -191,16 +203,16 @@ class AttentionPlan:
 
 
 def plan_for(head_dim: int, heads: int, kv_heads: int, distance_bias: bool = False, v_dim: Optional[int] = None,
-             softcap: float = 0.0, span: Optional[int] = None) -> Optional[AttentionPlan]:
+             softcap: float = 0.0, window: Optional[int] = None, chunk: Optional[int] = None) -> Optional[AttentionPlan]:
     if not supports(head_dim, v_dim) or (distance_bias and (softcap or (v_dim or head_dim) != head_dim)):
         return None
-    return AttentionPlan(head_dim, heads, kv_heads, distance_bias, v_dim, softcap, span)
+    return AttentionPlan(head_dim, heads, kv_heads, distance_bias, v_dim, softcap, window, chunk)
 
 
 def step_tiles(ctx, plan: AttentionPlan):
     """The step's row tiles for this head grouping: built once per step and shared by all layers."""
     key = ("attention_tiles", plan.group, plan.kv_heads, plan.head_dim, plan.distance_bias, plan.prefill_rows,
-           plan.decode is not None, plan.span)
+           plan.decode is not None, plan.window, plan.chunk)
     cached = ctx.extras.get(key)
     if cached is not None:
         return cached
@@ -216,6 +228,15 @@ def step_tiles(ctx, plan: AttentionPlan):
         h[at: at + c] = s
         h[n_tiles + at: n_tiles + at + c] = np.arange(c, dtype=np.int32)
         at += c
+    if plan.chunk and rows_per_tile != 16:
+        # the kernels start the last tile first: without blocks of positions it is the one that sees the most
+        # keys, with them the tiles are sorted by what they see
+        seq, index = h[:at].copy(), h[n_tiles: n_tiles + at].copy()
+        q_len, kv_len = np.asarray(ctx.host_q_len)[seq], np.asarray(ctx.host_kv_len)[seq]
+        first, last = index * rows_per_tile // g, np.minimum(((index + 1) * rows_per_tile - 1) // g, q_len - 1)
+        first, last = first + kv_len - q_len, last + kv_len - q_len
+        order = np.argsort(last - first // plan.chunk * plan.chunk, kind="stable")
+        h[:at], h[n_tiles: n_tiles + at] = seq[order], index[order]
     h[at: n_tiles] = -1
     h[n_tiles + at: 2 * n_tiles] = 0
     dev[: 2 * n_tiles].copy_(host[: 2 * n_tiles], non_blocking=True)
@@ -223,10 +244,9 @@ def step_tiles(ctx, plan: AttentionPlan):
     n_splits = 1
     use_decode = rows_per_tile == 16 and plan.decode is not None and n_tiles * plan.kv_heads <= DECODE_MAX_TILES
     if rows_per_tile == 16 and not use_decode:
-        key_blocks = -(-ctx.max_kv_len // KEY_BLOCK)
-        if plan.span:      # a tile's rows see `span` keys each, at most max_q_len positions apart
-            key_blocks = min(key_blocks, -(-(plan.span + ctx.max_q_len) // KEY_BLOCK) + 1)
+        key_blocks = plan.key_blocks(ctx.max_kv_len, ctx.max_q_len, KEY_BLOCK)
         n_splits = max(1, min(key_blocks, -(-(2 * sm_count()) // (n_tiles * plan.kv_heads))))
+        n_splits = -(-key_blocks // -(-key_blocks // n_splits))      # as many as the blocks per split leave busy
         if os.environ.get("BARE_CUDA_B200_ATTN_SPLITS"):     # experiments only
             n_splits = min(key_blocks, int(os.environ["BARE_CUDA_B200_ATTN_SPLITS"]))
         if n_tiles * plan.kv_heads > COUNTER_WORDS:
@@ -241,7 +261,9 @@ def step_tiles(ctx, plan: AttentionPlan):
         # on the context length (a short context leaves some warps without a key block), so a captured
         # graph of the step stays valid while the requests grow.
         dec_splits = 1
-        while dec_splits < 8 and n_tiles * plan.kv_heads * dec_splits * 2 <= 2 * sm_count():
+        # where a window or a block of positions bounds the keys: no more blocks of four warps than have a key block each
+        most = plan.key_blocks(1 << 30, ctx.max_q_len, plan.decode.key_block)
+        while dec_splits < 8 and 4 * dec_splits < most and n_tiles * plan.kv_heads * dec_splits * 2 <= 2 * sm_count():
             dec_splits *= 2
         dec_slots = 1
         if os.environ.get("BARE_CUDA_B200_ATTN_SPLITS"):     # experiments only

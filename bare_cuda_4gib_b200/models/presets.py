@@ -143,7 +143,7 @@ def _fuzazen(width, vocab, ff, heads, kv_heads, dim, vdim, chunk, rot_dims, own,
 
 
 PRESETS.update({
-    "fuzazen-tiny": _fuzazen(64, 300, 96, 4, 2, 16, 24, 20, 8, 2, 1),
+    "fuzazen-tiny": _fuzazen(64, 300, 96, 4, 2, 16, 32, 20, 8, 2, 1),
     # layer sizes of TinyLlama (width 2048, feed-forward 5632, 32 heads of 64, 4 key heads), blocks of 1,024 positions
     "fuzazen-2048": _fuzazen(2048, 32000, 5632, 32, 4, 64, 64, 1024, 64, 4, 1),
     # ... and of Llama-2-7B (width 4096, feed-forward 11008, 32 heads of 128)

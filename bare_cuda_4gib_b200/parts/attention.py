@@ -318,7 +318,7 @@ class GeneralAttention(Part):
             # equal head sizes without a cap: the engine's tcgen05 prefill, cluster decode and mma.sync kernels;
             # otherwise the mma.sync kernel built for this value size and with the cap (sizes it takes)
             from ..kernels import attention as fast
-            self.fast = fast.plan_for(self.dim, self.heads, self.kv_heads, False, self.vdim, self.softcap, self._span())
+            self.fast = fast.plan_for(self.dim, self.heads, self.kv_heads, False, self.vdim, self.softcap, self.window, self.chunk)
 
     def plan_step(self, ctx) -> None:
         if self.fast is not None and ctx.use_fast_attention:
