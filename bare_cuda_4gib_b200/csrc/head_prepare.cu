@@ -101,9 +101,11 @@ headnorm_rope_cache_kernel(const T* __restrict__ u, long long u_stride, int q_co
 }
 
 // The same with 16-byte accesses: bfloat16, neighbouring pairs, no bias and no value mixing, heads of 8, 16, 32,
-// 64, 128 or 256 entries.  A thread holds eight entries of a head (four pairs), so `d / 8` neighbouring lanes
-// of a warp hold a head and sum its squares among themselves; cos and sin are formed once per block and
-// pair instead of once per head.  Grid (token, share of the token's pieces).
+// 64, 128 or 256 entries.  A thread holds eight entries of a head (four pairs), so LANES = d / 8 neighbouring
+// lanes of a warp hold a head and sum its squares among themselves; cos and sin are formed once per block and
+// pair instead of once per head, while a thread's first piece is on its way, and every later piece is asked
+// for one round ahead.  Grid (token, share of the token's pieces).
+template <int LANES>
 __global__ void __launch_bounds__(PREP_WARPS * 32)
 headnorm_rope_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, int q_col, int k_col, int v_col,
                                const __nv_bfloat16* __restrict__ q_norm_w, const __nv_bfloat16* __restrict__ k_norm_w,
@@ -113,54 +115,63 @@ headnorm_rope_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_
                                int write_cache) {
   pdl_launch_dependents();
   pdl_wait();
+  constexpr int d = LANES * 8;
   __shared__ float2 turn[128];       // cos and sin of the token's angles, times mag
-  const int t = blockIdx.x, d = cache.head_dim, lanes = d / 8;
-  const int pos = positions[t], seq = row_seq[t];
+  const int t = blockIdx.x;
+  const int pos = positions[t];
+  const int q_pieces = q_heads * LANES, turned = q_pieces + cache.kv_heads * LANES;   // pieces of q, of q and k; then those of v
+  const int v_lanes = v_dim / 8, pieces = turned + (write_cache ? cache.kv_heads * v_lanes : 0);
+  const __nv_bfloat16* row = u + (long long)t * u_stride;
+  const uint4* q_row = reinterpret_cast<const uint4*>(row + q_col);
+  const uint4* k_row = reinterpret_cast<const uint4*>(row + k_col);
+  const uint4* v_row = reinterpret_cast<const uint4*>(row + (v_col >= 0 ? v_col : k_col));
+  auto piece = [&](int w) {          // heads and pieces lie side by side in the projection's row
+    return w < q_pieces ? q_row[w] : (w < turned ? k_row[w - q_pieces] : (w < pieces ? v_row[w - turned] : make_uint4(0, 0, 0, 0)));
+  };
+  const int step = gridDim.y * blockDim.x;
+  int w = blockIdx.y * blockDim.x + threadIdx.x;
+  uint4 next = piece(w);
   for (int p = threadIdx.x; p < rot_dims / 2; p += blockDim.x) {
     float sn, cs;
     sincosf((float)pos * inv_freq[p], &sn, &cs);
     turn[p] = make_float2(cs * mag, sn * mag);
   }
+  const int page = write_cache ? cache.block_table[(long long)row_seq[t] * cache.table_stride + pos / cache.page_tokens] : -1;
+  const int in_page = pos % cache.page_tokens;
+  __nv_bfloat16* k_page = (__nv_bfloat16*)cache.k + (long long)page * cache.page_stride;
+  __nv_bfloat16* v_page = (__nv_bfloat16*)cache.v + (long long)page * cache.page_stride;
   __syncthreads();
-  const int page = write_cache ? cache.block_table[(long long)seq * cache.table_stride + pos / cache.page_tokens] : -1;
-  const long long in_page = pos % cache.page_tokens;
-  const __nv_bfloat16* row = u + (long long)t * u_stride;
-  const int turned = (q_heads + cache.kv_heads) * lanes;                       // pieces of q and k, then those of v
-  const int pieces = turned + (page >= 0 ? cache.kv_heads * (v_dim / 8) : 0);
   // whole warps walk on together: a head's lanes lie in one warp and meet in its shuffles
-  for (int base = (blockIdx.y * blockDim.x + threadIdx.x) & ~31; base < pieces; base += gridDim.y * blockDim.x) {
-    const int w = base + (threadIdx.x & 31);
-    const bool is_qk = w < turned;
-    const int head = is_qk ? w / lanes : 0, part = is_qk ? w - head * lanes : 0;
-    const bool is_q = head < q_heads;
-    float x[8];
-    float sq = 0.0f;
-    if (is_qk) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(row + (is_q ? q_col + head * d : k_col + (head - q_heads) * d) + part * 8);
-      const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&raw);
+  for (; (w & ~31) < pieces; w += step) {
+    const uint4 raw = next;
+    next = piece(w + step);
+    const bool is_q = w < q_pieces;
+    if ((w & ~31) < turned) {
+      const __nv_bfloat162* e = reinterpret_cast<const __nv_bfloat162*>(&raw);
+      float2 x[4];
+      float sq = 0.0f;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        x[j] = __bfloat162float(e[j]);
-        sq += x[j] * x[j];
+      for (int j = 0; j < 4; ++j) {
+        x[j] = __bfloat1622float2(e[j]);
+        sq += x[j].x * x[j].x + x[j].y * x[j].y;
       }
-    }
-    for (int o = lanes / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-    if (is_qk) {
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
       const __nv_bfloat16* nw = is_q ? q_norm_w : k_norm_w;
-      const float scale = nw || unit_norm ? 1.0f / sqrtf(sq / (float)d + eps) : 1.0f;
-#pragma unroll
-      for (int j = 0; j < 8; ++j) x[j] *= scale;
-      if (nw) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(nw + part * 8);
-        const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&raw);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) x[j] *= __bfloat162float(e[j]);
-      }
-      uint4 packed;
+      const int part = w & (LANES - 1);
+      const float scale = nw || unit_norm ? 1.0f / sqrtf(sq * (1.0f / d) + eps) : 1.0f;
+      uint4 packed, wraw = make_uint4(0, 0, 0, 0);
+      if (nw) wraw = *reinterpret_cast<const uint4*>(nw + part * 8);
+      const __nv_bfloat162* we = reinterpret_cast<const __nv_bfloat162*>(&wraw);
       __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        float a = x[2 * j], b = x[2 * j + 1];
+        float a = x[j].x * scale, b = x[j].y * scale;
+        if (nw) {
+          const float2 f = __bfloat1622float2(we[j]);
+          a *= f.x;
+          b *= f.y;
+        }
         if (part * 8 + 2 * j < rot_dims) {
           const float2 cs = turn[part * 4 + j];
           const float na = a * cs.x - b * cs.y;
@@ -169,17 +180,16 @@ headnorm_rope_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_
         }
         o2[j] = __floats2bfloat162_rn(a, b);
       }
-      __nv_bfloat16* dst = nullptr;
-      if (is_q)
-        dst = q_out + ((long long)t * q_heads + head) * d;
-      else if (page >= 0)
-        dst = (__nv_bfloat16*)cache.k + (long long)page * cache.page_stride + ((long long)(head - q_heads) * cache.page_tokens + in_page) * d;
-      if (dst) *reinterpret_cast<uint4*>(dst + part * 8) = packed;
-    } else if (w < pieces) {
-      const int v = w - turned, g = v / (v_dim / 8), c = (v - g * (v_dim / 8)) * 8;
-      *reinterpret_cast<uint4*>((__nv_bfloat16*)cache.v + (long long)page * cache.page_stride +
-                                ((long long)g * cache.page_tokens + in_page) * v_dim + c) =
-          *reinterpret_cast<const uint4*>(row + (v_col >= 0 ? v_col : k_col) + g * v_dim + c);
+      if (is_q) {
+        reinterpret_cast<uint4*>(q_out + (long long)t * q_heads * d)[w] = packed;
+      } else if (w < turned && page >= 0) {
+        const int head = (w - q_pieces) / LANES;
+        *reinterpret_cast<uint4*>(k_page + ((long long)head * cache.page_tokens + in_page) * d + part * 8) = packed;
+      }
+    }
+    if (w >= turned && w < pieces && page >= 0) {
+      const int v = w - turned, g = v / v_lanes;
+      *reinterpret_cast<uint4*>(v_page + ((long long)g * cache.page_tokens + in_page) * v_dim + (v - g * v_lanes) * 8) = raw;
     }
   }
 }
@@ -211,10 +221,20 @@ extern "C" int llm_headnorm_rope_cache(const void* u, int dtype, long long u_str
     const int pieces = (q_heads + kv_heads) * (head_dim / 8) + kv_heads * (v_dim / 8);
     // few tokens: a token's pieces are dealt to several blocks
     const int shares = n_tokens >= 256 ? 1 : (pieces + PREP_WARPS * 32 - 1) / (PREP_WARPS * 32);
-    launch_kernel(headnorm_rope_cache_vec_kernel, dim3(n_tokens, shares < 16 ? shares : 16), PREP_WARPS * 32, 0, stream,
-                  (const __nv_bfloat16*)u, u_stride, q_col, k_col, v_col, (const __nv_bfloat16*)q_norm_w,
-                  (const __nv_bfloat16*)k_norm_w, unit_norm, eps, inv_freq, rot_dims, mag, (__nv_bfloat16*)q_out, c, v_dim,
-                  positions, row_seq, q_heads, write_cache);
+    const dim3 grid(n_tokens, shares < 16 ? shares : 16);
+#define LAUNCH_VEC(LANES)                                                                                              \
+  launch_kernel(headnorm_rope_cache_vec_kernel<LANES>, grid, PREP_WARPS * 32, 0, stream, (const __nv_bfloat16*)u,      \
+                u_stride, q_col, k_col, v_col, (const __nv_bfloat16*)q_norm_w, (const __nv_bfloat16*)k_norm_w, unit_norm, \
+                eps, inv_freq, rot_dims, mag, (__nv_bfloat16*)q_out, c, v_dim, positions, row_seq, q_heads, write_cache)
+    switch (head_dim) {
+      case 8: LAUNCH_VEC(1); break;
+      case 16: LAUNCH_VEC(2); break;
+      case 32: LAUNCH_VEC(4); break;
+      case 64: LAUNCH_VEC(8); break;
+      case 128: LAUNCH_VEC(16); break;
+      default: LAUNCH_VEC(32); break;
+    }
+#undef LAUNCH_VEC
     return launch_status();
   }
   // few tokens: a token's heads are dealt to several blocks, so that the step still fills the GPU
