@@ -12,6 +12,7 @@
 #include <math.h>
 
 #define NORM_THREADS 256
+#define FEW_ROWS 64
 
 template <typename TT, typename TW>
 __global__ void __launch_bounds__(NORM_THREADS)
@@ -105,16 +106,19 @@ postnorm_add_rmsnorm_kernel(float* __restrict__ residual, const float* __restric
     dst[i] = from_float<TO>(row_cache[i] * s2 * to_float(next_w[i]));
 }
 
-// The same with 16-byte accesses for bfloat16 weights and output: width a multiple of 4 up to 16 x the
+// The same with 16-byte accesses for bfloat16 weights and output: width a multiple of 4 up to 4 x HOLD x the
 // block size, every row's pieces in registers (a thread's sums are formed in another order than
-// the kernel above forms them: float32 rounding under a bfloat16 result).
+// the kernel above forms them: float32 rounding under a bfloat16 result).  HOLD pieces a thread in blocks of
+// NORM_THREADS for many rows; for few rows (a decode step, whose results may be many partial sums) one piece a
+// thread in blocks as wide as the row, so that a row's loads are in flight together.
 __device__ __forceinline__ float4 bf16x4(const __nv_bfloat16* p) {
   const uint2 raw = *reinterpret_cast<const uint2*>(p);
   const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), b = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
   return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
 }
 
-__global__ void __launch_bounds__(NORM_THREADS)
+template <int HOLD>
+__global__ void __launch_bounds__(HOLD == 1 ? 1024 : NORM_THREADS)
 postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __restrict__ y, int n_partials,
                                 long long partial_stride, const __nv_bfloat16* __restrict__ post_w, float post_eps, float mult,
                                 const __nv_bfloat16* __restrict__ next_w, float next_eps, __nv_bfloat16* __restrict__ out,
@@ -126,14 +130,15 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
   const long long src = row_index ? row_index[r] : r;
   float4* x = reinterpret_cast<float4*>(residual + src * hidden);
   const int n4 = hidden / 4;
-  float4 v[4], old[4];
+  float4 v[HOLD], old[HOLD];
   float sq = 0.0f;
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = threadIdx.x + j * NORM_THREADS;
+  for (int j = 0; j < HOLD; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
     if (i < n4) {
       old[j] = x[i];
       float4 a = y ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : old[j];
+#pragma unroll 4
       for (int p = 0; p < n_partials; ++p) {
         const float4 d = reinterpret_cast<const float4*>(y + p * partial_stride + src * hidden)[i];
         a.x += d.x; a.y += d.y; a.z += d.z; a.w += d.w;
@@ -146,8 +151,8 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
     const float s1 = mult / sqrtf(block_sum(sq, scratch) / (float)hidden + post_eps);
     sq = 0.0f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = threadIdx.x + j * NORM_THREADS;
+    for (int j = 0; j < HOLD; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
       if (i < n4) {
         const float4 w = bf16x4(post_w + 4 * i);
         float4 a = old[j];
@@ -162,8 +167,8 @@ postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, const float* __res
   const float s2 = next_w ? 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + next_eps) : 1.0f;
   uint2* dst = reinterpret_cast<uint2*>(out + (long long)r * hidden);
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = threadIdx.x + j * NORM_THREADS;
+  for (int j = 0; j < HOLD; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
     if (i < n4) {
       const float4 w = next_w ? bf16x4(next_w + 4 * i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
       const __nv_bfloat162 lo = __floats2bfloat162_rn(v[j].x * s2 * w.x, v[j].y * s2 * w.y);
@@ -193,10 +198,17 @@ extern "C" int llm_postnorm_add_rmsnorm(float* residual, const float* y, int n_p
                   hidden);
   else if (dtype == DT_BF16 && hidden % 4 == 0 && hidden <= 16 * NORM_THREADS && partial_stride % 4 == 0 &&
            ((uintptr_t)residual % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)post_w % 8) == 0 &&
-           ((uintptr_t)next_w % 8) == 0 && ((uintptr_t)out % 8) == 0)
-    launch_kernel(postnorm_add_rmsnorm_vec_kernel, rows, NORM_THREADS, 0, stream, residual, y, n_partials, partial_stride,
-                  (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w, next_eps, (__nv_bfloat16*)out,
-                  row_index, hidden);
+           ((uintptr_t)next_w % 8) == 0 && ((uintptr_t)out % 8) == 0) {
+    const int wide = rows > FEW_ROWS ? 0 : (hidden + 127) / 128 * 32;      // threads that hold a row, one piece each
+    if (wide > NORM_THREADS && wide <= 1024)
+      launch_kernel(postnorm_add_rmsnorm_vec_kernel<1>, rows, wide, 0, stream, residual, y, n_partials, partial_stride,
+                    (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w, next_eps, (__nv_bfloat16*)out,
+                    row_index, hidden);
+    else
+      launch_kernel(postnorm_add_rmsnorm_vec_kernel<4>, rows, NORM_THREADS, 0, stream, residual, y, n_partials,
+                    partial_stride, (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w, next_eps,
+                    (__nv_bfloat16*)out, row_index, hidden);
+  }
   else if (dtype == DT_BF16)
     launch_kernel(postnorm_add_rmsnorm_kernel<__nv_bfloat16, __nv_bfloat16>, rows, NORM_THREADS, smem, stream, residual,
                   y, n_partials, partial_stride, (const __nv_bfloat16*)post_w, post_eps, mult, (const __nv_bfloat16*)next_w,

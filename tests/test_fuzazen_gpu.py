@@ -205,13 +205,13 @@ def test_long_prompts_in_blocks():
         _close(got, want, 1.5e-2)
 
 
-@pytest.mark.parametrize("width", [52, 256, 50, 6000])
+@pytest.mark.parametrize("n", [9, 90])
+@pytest.mark.parametrize("width", [52, 256, 50, 1100, 2048, 4096, 6000])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_stream_kernels(dtype, width):
+def test_stream_kernels(dtype, width, n):
     """x + m * rms_norm(y) * w with the new stream handed on un-normed, and the stream alone."""
     from bare_cuda_4gib_b200.kernels import lib as K, sandwich as SW
     g = torch.Generator().manual_seed(4)
-    n = 9
     x = torch.randn(n, width, generator=g)
     y = torch.randn(3, n, width, generator=g)                # three partial sums
     w = torch.randn(width, generator=g).to(dtype)
