@@ -159,8 +159,21 @@ struct DecodeArgs {
   int* error_word;
 };
 
+// Clears the value rows from `first` on of a key block at `v_base` (one warp).
+__device__ __noinline__ void clear_value_rows(uint32_t v_base, int first, int lane) {
+  for (int i = lane; i < (BN - first) * SUBS * 8; i += 32) {
+    const int r = first + i / (SUBS * 8), c = i % (SUBS * 8);
+    asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(v_base + (c / 8) * SUB_BYTES + r * 128 + (c % 8) * 16), "r"(0) : "memory");
+  }
+  __syncwarp();
+}
+
+// EXTRAS: whether blocks of positions, a sink or a gate may be asked for; without them their code is not there.
+template <bool EXTRAS>
 __global__ void __launch_bounds__(THREADS)
 attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const DecodeArgs a) {
+  const AttentionExtras extras = EXTRAS ? a.extras : AttentionExtras{0, nullptr, nullptr, 0};
+  const int window = a.window;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* kv = smem;                                                       // [WARPS][slots][KV_BYTES]
@@ -204,8 +217,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
   const int last_token = min(q_len - 1, (row0 + BM - 1) / group), first_token = row0 / group;
   const int hi_key = pos0 + last_token;
   const int tile_min_pos = pos0 + first_token, tile_max_pos = pos0 + last_token;
-  const int lo_key = first_visible_key(tile_min_pos, a.window, a.extras.chunk);
-  const int tile_max_lo = first_visible_key(tile_max_pos, a.window, a.extras.chunk);   // from here on no row's bound hides a key
+  const int lo_key = first_visible_key(tile_min_pos, window, extras.chunk);
+  const int tile_max_lo = first_visible_key(tile_max_pos, window, extras.chunk);   // from here on no row's bound hides a key
   const int kb_lo = lo_key / BN, kb_hi = hi_key / BN;   // inclusive
   // this warp's key blocks: kb_lo + gw, kb_lo + gw + stride, ...
   const int stride = WARPS * n_splits, gw = split * WARPS + warp;
@@ -290,7 +303,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
   for (int h = 0; h < 2; ++h) {
     const int R = row0 + (lane >> 2) + h * 8;
     row_pos[h] = R < n_rows ? pos0 + R / group : -1;
-    row_lo[h] = first_visible_key(row_pos[h], a.window, a.extras.chunk);
+    row_lo[h] = first_visible_key(row_pos[h], window, extras.chunk);
     m[h] = -INFINITY;
     l[h] = 0.0f;
   }
@@ -304,15 +317,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
     const uint32_t k_base = smem_u32(my_kv) + slot * KV_BYTES, v_base = k_base + SUBS * SUB_BYTES;
     const int kb = kb_lo + gw + j * stride;
     const int key0 = kb * BN;
-    if (key0 + BN > kv_len) {
-      // the request's last key block: a page may hold anything behind the last key, and a weight of zero
-      // times NaN is not zero, so those value rows are cleared (no later block of this warp uses the slot)
-      for (int i = lane; i < (key0 + BN - kv_len) * SUBS * 8; i += 32) {
-        const int r = kv_len - key0 + i / (SUBS * 8), c = i % (SUBS * 8);
-        asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(v_base + (c / 8) * SUB_BYTES + r * 128 + (c % 8) * 16), "r"(0) : "memory");
-      }
-      __syncwarp();
-    }
+    // the request's last key block: a page may hold anything behind the last key, and a weight of zero times NaN
+    // is not zero, so those value rows are cleared here or (head size 128, where it
+    // measured faster) before the second product (no later block of this warp uses the slot)
+    if (D == 64 && __builtin_expect(key0 + BN > kv_len, 0)) clear_value_rows(v_base, kv_len - key0, lane);
 
     float s[NT][4];
 #pragma unroll
@@ -385,6 +393,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
       pf[nt / 2][(nt & 1) * 2 + 0] = pack_bf16(p0, p1);
       pf[nt / 2][(nt & 1) * 2 + 1] = pack_bf16(p2, p3);
     }
+    if (D != 64 && __builtin_expect(key0 + BN > kv_len, 0)) clear_value_rows(v_base, kv_len - key0, lane);
 #pragma unroll
     for (int kk = 0; kk < BN / 16; ++kk) {
       const int key = kk * 16 + (mid & 1) * 8 + (lane & 7);
@@ -462,7 +471,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
     const int r = slot * n_splits + split, R = row0 + r;
     if (r >= BM || R >= n_rows) continue;
     const int token = R / group, head = kvh * group + R % group;
-    const float sink = sink_log2(a.extras, head);     // joins the row's sum here, once
+    const float sink = sink_log2(extras, head);     // joins the row's sum here, once
     float M = sink;
     for (int z = 0; z < n_splits; ++z) M = fmaxf(M, recv[((size_t)z * owned_rows + slot) * STATE + D]);
     float L = M != -INFINITY ? exp2f(sink - M) : 0.0f;
@@ -479,7 +488,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap pool_map, const Deco
         acc.w += v.w * f;
       }
     }
-    const float inv = L > 0.0f ? head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / L : 0.0f;
+    const float inv = L > 0.0f ? head_gate<__nv_bfloat16>(extras, q_start + token, head) / L : 0.0f;
     uint2 packed;
     packed.x = pack_bf16(acc.x * inv, acc.y * inv);
     packed.y = pack_bf16(acc.z * inv, acc.w * inv);
@@ -557,7 +566,8 @@ extern "C" int llm_attention_decode(const void* pool_map, const void* pool_base,
   if (smem > 227 * 1024) return ERR_BAD_SIZE;
   static size_t raised = 0;
   if (smem > raised) {
-    if (cudaFuncSetAttribute(attention_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return launch_status();
     raised = smem;
   }
@@ -598,6 +608,6 @@ extern "C" int llm_attention_decode(const void* pool_map, const void* pool_base,
   }
   cfg.attrs = attr;
   cfg.numAttrs = n_attr;
-  cudaLaunchKernelEx(&cfg, attention_decode_kernel, map, a);
+  cudaLaunchKernelEx(&cfg, chunk > 0 || sink || gate ? attention_decode_kernel<true> : attention_decode_kernel<false>, map, a);
   return launch_status();
 }

@@ -132,9 +132,11 @@ __device__ __forceinline__ float capped_score(float raw, float scale_over_cap, f
   return cap_log2 * (1.0f - __fdividef(2.0f, t + 1.0f));
 }
 
-template <int WARPS_M, int WARPS_N, int MT>
+// EXTRAS: whether blocks of positions, a sink or a gate may be asked for; without them their code is not there.
+template <int WARPS_M, int WARPS_N, int MT, bool EXTRAS>
 __global__ void __launch_bounds__(WARPS_M* WARPS_N * 32)
 attention_mma_kernel(AttnArgs a) {
+  const AttentionExtras extras = EXTRAS ? a.extras : AttentionExtras{0, nullptr, nullptr, 0};
   constexpr int NW = WARPS_M * WARPS_N;
   constexpr int NT_THREADS = NW * 32;
   constexpr int WR = 16 * MT;            // rows per warp
@@ -172,8 +174,8 @@ attention_mma_kernel(AttnArgs a) {
   // (their queries are zero, their scores finite).
   const int tile_min_pos = pos0 + first_token;
   const int tile_max_pos = pos0 + last_token;
-  const int lo_key = first_visible_key(tile_min_pos, a.window, a.extras.chunk);
-  const int tile_max_lo = first_visible_key(tile_max_pos, a.window, a.extras.chunk);   // from here on no row's bound hides a key
+  const int lo_key = first_visible_key(tile_min_pos, a.window, extras.chunk);
+  const int tile_max_lo = first_visible_key(tile_max_pos, a.window, extras.chunk);   // from here on no row's bound hides a key
   const int kb_lo = lo_key / BN, kb_hi = hi_key / BN;  // inclusive
   const int n_kb_total = kb_hi - kb_lo + 1;
   const int per_split = (n_kb_total + n_splits - 1) / n_splits;
@@ -286,7 +288,7 @@ attention_mma_kernel(AttnArgs a) {
     for (int h = 0; h < 2; ++h) {
       const int R = row0 + wm * WR + mt * 16 + (lane >> 2) + h * 8;
       row_pos[mt][h] = R < n_rows ? pos0 + R / group : -1;  // -1: no key is visible
-      row_lo[mt][h] = first_visible_key(row_pos[mt][h], a.window, a.extras.chunk);
+      row_lo[mt][h] = first_visible_key(row_pos[mt][h], a.window, extras.chunk);
 #ifdef DISTANCE_BIAS
       row_bias[mt][h] = a.bias + (long long)(kvh * group + R % group) * a.bias_len;
 #endif
@@ -469,7 +471,7 @@ attention_mma_kernel(AttnArgs a) {
     const int R = row0 + r;
     const int token = R / group, head = kvh * group + R % group;
     // a row that is finished here (keys not split) has the sink in its sum from the start
-    const float sink = n_splits == 1 && R < n_rows ? sink_log2(a.extras, head) : -INFINITY;
+    const float sink = n_splits == 1 && R < n_rows ? sink_log2(extras, head) : -INFINITY;
     float M = sink;
 #pragma unroll
     for (int w = 0; w < WARPS_N; ++w) M = fmaxf(M, red_m[w * BM + r]);
@@ -486,7 +488,7 @@ attention_mma_kernel(AttnArgs a) {
     }
     if (n_splits == 1) {
       if (R < n_rows) {
-        const float inv = L > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / L : 0.0f;
+        const float inv = L > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(extras, q_start + token, head) / L : 0.0f;
         uint4 packed;
         packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
         packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
@@ -529,7 +531,7 @@ attention_mma_kernel(AttnArgs a) {
     if (R >= n_rows) continue;
     auto lse_at = [&](int z) { return lse_fits ? lse[z * BM + r] : __ldcg(a.part_lse + (item0 + z) * BM + r); };
     const int token = R / group, head = kvh * group + R % group;
-    const float sink = sink_log2(a.extras, head);
+    const float sink = sink_log2(extras, head);
     float M = sink;
     for (int z = 0; z < n_splits; ++z) M = fmaxf(M, lse_at(z));
     float W = M != -INFINITY ? exp2f(sink - M) : 0.0f, acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
@@ -544,7 +546,7 @@ attention_mma_kernel(AttnArgs a) {
         acc[4] += w * hi.x; acc[5] += w * hi.y; acc[6] += w * hi.z; acc[7] += w * hi.w;
       }
     }
-    const float inv = W > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(a.extras, q_start + token, head) / W : 0.0f;
+    const float inv = W > 0.0f ? a.out_scale * head_gate<__nv_bfloat16>(extras, q_start + token, head) / W : 0.0f;
     uint4 packed;
     packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
     packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
@@ -564,9 +566,9 @@ constexpr size_t smem_bytes() {
   return tiles > merge ? tiles : merge;
 }
 
-template <int WARPS_M, int WARPS_N, int MT>
-int launch(const AttnArgs& a, int n_tiles, int kv_heads, int n_splits, cudaStream_t stream) {
-  auto kern = attention_mma_kernel<WARPS_M, WARPS_N, MT>;
+template <int WARPS_M, int WARPS_N, int MT, bool EXTRAS>
+int launch_form(const AttnArgs& a, int n_tiles, int kv_heads, int n_splits, cudaStream_t stream) {
+  auto kern = attention_mma_kernel<WARPS_M, WARPS_N, MT, EXTRAS>;
   constexpr size_t smem = smem_bytes<WARPS_M, WARPS_N, MT>();
   static bool configured = false;
   if (!configured) {
@@ -578,6 +580,15 @@ int launch(const AttnArgs& a, int n_tiles, int kv_heads, int n_splits, cudaStrea
   dim3 grid(n_tiles, kv_heads, n_splits);
   launch_kernel(kern, grid, WARPS_M * WARPS_N * 32, smem, stream, a);
   return launch_status();
+}
+
+template <int WARPS_M, int WARPS_N, int MT>
+int launch(const AttnArgs& a, int n_tiles, int kv_heads, int n_splits, cudaStream_t stream) {
+#ifndef DISTANCE_BIAS      // that variant's entry point offers none of them
+  if (a.extras.chunk > 0 || a.extras.sink || a.extras.gate)
+    return launch_form<WARPS_M, WARPS_N, MT, true>(a, n_tiles, kv_heads, n_splits, stream);
+#endif
+  return launch_form<WARPS_M, WARPS_N, MT, false>(a, n_tiles, kv_heads, n_splits, stream);
 }
 
 }  // namespace

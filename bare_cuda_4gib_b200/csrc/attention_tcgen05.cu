@@ -218,8 +218,13 @@ struct AttnArgs {
 
 constexpr int ERR_LOADER = 11, ERR_MMA = 12, ERR_SOFTMAX = 13, ERR_LAYOUT = 14;
 
+// EXTRAS: whether a window, blocks of positions, a sink or a gate may be asked for; without them their code is
+// not there.
+template <bool EXTRAS>
 __global__ void __launch_bounds__(NUM_THREADS, TILES == 1 ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs a) {
+  const AttentionExtras extras = EXTRAS ? a.extras : AttentionExtras{0, nullptr, nullptr, 0};
+  const int window = EXTRAS ? a.window : 0;
   extern __shared__ __align__(1024) uint8_t smem[];   // swizzled tiles need 1024-byte alignment (checked below)
   uint8_t* q_smem = smem;                              // [TILES][KA sub-tiles]
   uint8_t* ring = q_smem + TILES * Q_BYTES;            // [SLOTS][KA sub-tiles]: key and value tiles in turn
@@ -269,7 +274,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
       const int first_token = first_row / group, last_token = min(q_len - 1, (first_row + BM - 1) / group);
       g_min_pos[g] = pos0 + first_token;
       g_max_pos[g] = pos0 + last_token;
-      const int lo_key = first_visible_key(g_min_pos[g], a.window, a.extras.chunk);
+      const int lo_key = first_visible_key(g_min_pos[g], window, extras.chunk);
       g_lo[g] = lo_key / BN;
       g_hi[g] = g_max_pos[g] / BN + 1;
       lo_all = min(lo_all, g_lo[g]);
@@ -438,13 +443,23 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
         for (int g = 0; g < TILES; ++g) any = any || pv_next[g] < n_g[g];
         return any;
       };
-      // Whether tile n has landed.  A barrier's parity tells one filling of a slot only from the one before it, so
-      // the tiles are counted off in order: a group whose first key block lies several blocks behind the
-      // other's (it begins in a later block of positions) would else take an earlier filling for its own.
-      int arrived = 0;
+      // Whether tile n has landed.  A barrier's parity tells one filling of a slot only from the one before it.
+      // Groups that start with the same key block ask for the tiles as the slots are filled.  A group whose
+      // first key block lies behind the other's (a window, or a later block of positions) would take an
+      // earlier filling for its own: there the tiles are counted off in order.
+      const bool counted = EXTRAS && TILES > 1 && g_lo[0] != g_lo[TILES - 1];
+      int arrived = 0, arrived_slot = 0;
+      uint32_t arrived_parity = 0;
       auto landed = [&](int n) {
-        while (arrived <= n && mbar_try_wait(&tile_full[arrived % SLOTS], (arrived / SLOTS) & 1)) ++arrived;
-        return arrived > n;
+        if (counted) {
+          while (arrived <= n) {
+            if (!mbar_try_wait(&tile_full[arrived_slot], arrived_parity)) return false;
+            ++arrived;
+            if (++arrived_slot == SLOTS) arrived_slot = 0, arrived_parity ^= 1u;
+          }
+          return true;
+        }
+        return mbar_try_wait(&tile_full[n % SLOTS], (n / SLOTS) & 1);
       };
       unsigned long long idle_since = 0;
       unsigned idle_spins = 0;
@@ -514,9 +529,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
     const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
     const uint32_t s_addr = lane_addr + g * BN, o_addr = lane_addr + O_COL + g * D;
     const int my_lo = g_lo[g], my_n = g_hi[g] - g_lo[g];
-    const int row_lo = first_visible_key(row_pos, a.window, a.extras.chunk);
+    const int row_lo = first_visible_key(row_pos, window, extras.chunk);
     const int tile_min_pos = g_min_pos[g];
-    const int tile_max_lo = first_visible_key(g_max_pos[g], a.window, a.extras.chunk);   // from here on no row's bound hides a key
+    const int tile_max_lo = first_visible_key(g_max_pos[g], window, extras.chunk);   // from here on no row's bound hides a key
     // Running softmax of the row.  `m` is the maximum the exponentials are taken against; it follows the
     // true maximum only when that has grown by more than RESCALE_STEP (in base-2 units), so that O, which
     // accumulates in tensor memory over all key blocks, has to be rescaled rarely: with a stale maximum
@@ -534,7 +549,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
       ok = mbar_wait(&s_full[g], i & 1, abort_flag) && !*abort_flag;
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const bool all_visible = key0 + BN - 1 <= tile_min_pos && key0 >= tile_max_lo;
+      const bool all_visible = key0 + BN - 1 <= tile_min_pos && (!EXTRAS || key0 >= tile_max_lo);
       // The row of S is read once, in two pieces of 64 columns (one sub-tile of P each).  Each piece
       // settles the maximum for itself: should the second piece move it, the probabilities of the
       // first, which this thread has just written, are rescaled where they lie (rare, as is every move).
@@ -553,7 +568,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
 #pragma unroll
           for (int k = 0; k < S_PIECE; ++k) {
             const int key = key0 + h * S_PIECE + k;
-            const bool visible = key <= row_pos && key >= row_lo;
+            const bool visible = key <= row_pos && (!EXTRAS || key >= row_lo);
             if (!visible) v[k] = 0xff800000u;   // -inf: probability 0
           }
         }
@@ -645,8 +660,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap pool_map, AttnArgs 
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int token = row_valid ? R / group : 0, head = row_valid ? kvh * group + R % group : 0;
       // the sink joins the sum, taken against the same maximum (far above it the sum is infinite, the row zero)
-      if (a.extras.sink && row_valid) l += exp2f(sink_log2(a.extras, head) - m);
-      const float inv = l > 0.0f ? (row_valid ? head_gate<__nv_bfloat16>(a.extras, q_start + token, head) : 1.0f) / l : 0.0f;
+      if (extras.sink && row_valid) l += exp2f(sink_log2(extras, head) - m);
+      const float inv = l > 0.0f ? (row_valid ? head_gate<__nv_bfloat16>(extras, q_start + token, head) : 1.0f) / l : 0.0f;
       uint4* dst = reinterpret_cast<uint4*>(a.out + ((long long)(q_start + token) * a.q_heads + head) * D);
 #pragma unroll
       for (int c0 = 0; c0 < D; c0 += 32) {
@@ -732,8 +747,10 @@ extern "C" int llm_attention_tcgen05(const void* pool_map, const void* pool_base
     return ERR_BAD_ALIGN;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES) !=
-        cudaSuccess)
+    if (cudaFuncSetAttribute(attention_tcgen05_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES) !=
+            cudaSuccess ||
+        cudaFuncSetAttribute(attention_tcgen05_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES) !=
+            cudaSuccess)
       return launch_status();
     configured = true;
   }
@@ -759,6 +776,7 @@ extern "C" int llm_attention_tcgen05(const void* pool_map, const void* pool_base
   a.error_word = error_word;
   if (n_tiles > 65535) return ERR_BAD_SIZE;
   dim3 grid(kv_heads, n_tiles);
-  launch_kernel(attention_tcgen05_kernel, grid, NUM_THREADS, SMEM_BYTES, stream, map, a);
+  launch_kernel(window > 0 || chunk > 0 || sink || gate ? attention_tcgen05_kernel<true> : attention_tcgen05_kernel<false>, grid,
+                NUM_THREADS, SMEM_BYTES, stream, map, a);
   return launch_status();
 }
