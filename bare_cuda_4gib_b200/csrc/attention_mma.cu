@@ -361,7 +361,8 @@ attention_mma_kernel(AttnArgs a) {
           for (int e = 0; e < 4; ++e) {
             const int h = e >> 1;
             const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-            const bool visible = key <= row_pos[mt][h] && key >= row_lo[mt][h];
+            const bool visible = key <= row_pos[mt][h] &&
+                                 (EXTRAS ? key >= row_lo[mt][h] : a.window <= 0 || key > row_pos[mt][h] - a.window);
 #ifdef DISTANCE_BIAS
             const float v = visible ? fmaf(s[mt][nt][e], a.scale_log2,
                                            1.4426950408889634f * __ldg(row_bias[mt][h] + min(row_pos[mt][h] - key, a.bias_len - 1)))

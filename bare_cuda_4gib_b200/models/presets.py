@@ -139,7 +139,7 @@ def _fuzazen(width, vocab, ff, heads, kv_heads, dim, vdim, chunk, rot_dims, own,
     for _ in range(repeats):
         layers = layers + [dict(layer, weights_of=j) for j in range(own)]
     return dict(architecture="Fuzazen", vocab=vocab, width=width, embedding={"scale": 1.0}, norm={"eps": 1e-6},
-                residual_mult=0.5, logit_softcap=30.0, layers=layers)
+                residual_mult=0.6, logit_softcap=50.0, layers=layers)
 
 
 PRESETS.update({

@@ -26,7 +26,7 @@ def again(layer, j):
     return dict(copy.deepcopy(layer), weights_of=j)
 
 
-def model(layers, width, vocab, scale=1.0, mult=0.5, cap=30.0, eps=1e-5):
+def model(layers, width, vocab, scale=1.3, mult=0.6, cap=25.0, eps=1e-5):
     return {"architecture": "Fuzazen", "vocab": vocab, "width": width, "embedding": {"scale": scale}, "norm": {"eps": eps},
             "residual_mult": mult, "logit_softcap": cap, "layers": copy.deepcopy(layers)}
 

@@ -57,7 +57,7 @@ ALONE = {
     "tight_cap": ([U.attention(2, 1, 32, 16, 25, 16, ff=40)], dict(cap=1.0, mult=2.0)),
     "no_cap": ([U.attention(2, 1, 32, 16, 25, 16)], dict(cap=None)),
     "width_50": ([U.attention(3, 3, 12, 20, 17, 6, ff=34)], dict(width=50)),        # nothing lines up with 16 bytes
-    "width_256": ([U.attention(6, 2, 64, 32, 60, 40, scale=0.15, ff=320)], dict(width=256)),
+    "width_192": ([U.attention(9, 3, 64, 32, 60, 40, scale=0.15, ff=288)], dict(width=192)),
 }
 
 
