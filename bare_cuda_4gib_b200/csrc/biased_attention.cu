@@ -5,6 +5,7 @@
 //     inputs per request are kept in a state slot as a ring indexed by position;
 //   * an RMS norm over the whole q projection and over the whole k projection (all heads at once);
 //   * a factor on q that grows with the logarithm of the position;
+//   * a rotation by position of a head's first entries of q and k, in neighbouring pairs or in halves;
 //   * a bias per (distance, head) added to the scaled score, read from a table by distance;
 //   * key and value heads of different sizes.
 //
@@ -39,7 +40,9 @@ __device__ __forceinline__ int cache_page(const PagedCacheKV& c, int seq, int po
 //   y[c] = sum_j w[c][j] * U(p - taps + 1 + j)[c],  U(x) = 0 for x < 0, the step's own row for
 //   x >= p0, and the ring entry x % (taps - 1) of the request's state otherwise.
 // Then q = y_q / rms(y_q) * wq * (1 + coef * ln(floor((p + 1) / every) + 1)), k = y_k / rms(y_k) * wk,
-// v = y_v; q goes to q_out, k and v into the cache.
+// v = y_v; with `inv_freq` the first `rot_dims` entries of every q and k head are turned pair by pair (entry
+// 2i with 2i + 1, or with `halves` i with i + rot_dims / 2) by the angle p * inv_freq[i]; q goes to q_out, k
+// and v into the cache.
 template <typename T>
 __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restrict__ u, long long u_stride, const float* __restrict__ conv_w,
                                        int taps, const float* __restrict__ ring, const float* __restrict__ q_norm_w,
@@ -47,11 +50,12 @@ __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restric
                                        const int32_t* __restrict__ positions, const int32_t* __restrict__ row_seq,
                                        const int32_t* __restrict__ seq_slot, const int32_t* __restrict__ seq_q_start,
                                        int qd, int kd, int vd, float eps, float temp_coef, int temp_every,
-                                       int write_cache) {
+                                       int write_cache, const float* __restrict__ inv_freq, int rot_dims, int halves) {
   pdl_launch_dependents();
-  extern __shared__ float ys[];      // C floats + 32 scratch
+  extern __shared__ float ys[];      // C floats + 32 scratch + rot_dims cosines and sines
   const int C = qd + kd + vd;
   float* scratch = ys + C;
+  float* turn = scratch + 32;        // [rot_dims / 2] cosines, then as many sines
   pdl_wait();
   const int t = blockIdx.x;
   const int seq = row_seq[t], p = positions[t];
@@ -81,21 +85,33 @@ __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restric
     if (c < qd) sq_q += y * y;
     else if (c < qd + kd) sq_k += y * y;
   }
-  const float tq = block_sum(sq_q, scratch);
+  const int half = inv_freq ? rot_dims / 2 : 0;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)p * inv_freq[i], &turn[half + i], &turn[i]);
+  const float tq = block_sum(sq_q, scratch);      // (its barriers also make ys and turn whole)
   const float tk = block_sum(sq_k, scratch);
   const float rq = 1.0f / sqrtf(tq / (float)qd + eps) * (1.0f + temp_coef * logf((float)((p + 1) / temp_every + 1)));
   const float rk = 1.0f / sqrtf(tk / (float)kd + eps);
   const int page = cache_page(cache, seq, p);
   const int in_page = p % cache.page_tokens;
-  const int G = cache.kv_heads;
+  // entry d of a head whose channels start at c0: normed, and turned where the rotation reaches
+  auto head_entry = [&](int c0, int d, float r, const float* w) -> float {
+    const float v = ys[c0 + d] * r * w[d];
+    if (d >= 2 * half) return v;
+    const int i = halves ? (d < half ? d : d - half) : d >> 1;
+    const bool second = halves ? d >= half : d & 1;
+    const int e = halves ? (second ? d - half : d + half) : d ^ 1;
+    const float other = ys[c0 + e] * r * w[e];
+    return second ? v * turn[i] + other * turn[half + i] : v * turn[i] - other * turn[half + i];
+  };
   for (int c = threadIdx.x; c < C; c += blockDim.x) {
     if (c < qd) {
-      q_out[(long long)t * qd + c] = from_float<T>(ys[c] * rq * q_norm_w[c]);
+      const int d = c % cache.k_dim;
+      q_out[(long long)t * qd + c] = from_float<T>(head_entry(c - d, d, rq, q_norm_w + (c - d)));
     } else if (write_cache && page >= 0) {
       if (c < qd + kd) {
         const int e = c - qd, g = e / cache.k_dim, d = e - g * cache.k_dim;
         T* dst = (T*)cache.k + (long long)page * cache.page_stride + ((long long)g * cache.page_tokens + in_page) * cache.k_dim + d;
-        *dst = from_float<T>(ys[c] * rk * k_norm_w[e]);
+        *dst = from_float<T>(head_entry(c - d, d, rk, k_norm_w + (e - d)));
       } else {
         const int e = c - qd - kd, g = e / cache.v_dim, d = e - g * cache.v_dim;
         T* dst = (T*)cache.v + (long long)page * cache.page_stride + ((long long)g * cache.page_tokens + in_page) * cache.v_dim + d;
@@ -103,7 +119,6 @@ __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restric
       }
     }
   }
-  (void)G;
 }
 
 extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride, const float* conv_w, int taps,
@@ -112,12 +127,15 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
                                    int table_stride, int page_tokens, int kv_heads, int k_dim, int v_dim,
                                    const int32_t* positions, const int32_t* row_seq, const int32_t* seq_slot,
                                    const int32_t* seq_q_start, int n_tokens, int q_heads, float eps, float temp_coef,
-                                   int temp_every, int write_cache, cudaStream_t stream) {
+                                   int temp_every, int write_cache, const float* inv_freq, int rot_dims, int halves,
+                                   cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   LLM_HOST_CHECK(taps >= 1 && temp_every >= 1, ERR_BAD_SIZE);
+  if (!inv_freq) rot_dims = 0;
+  LLM_HOST_CHECK(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= k_dim, ERR_BAD_SIZE);
   const int qd = q_heads * k_dim, kd = kv_heads * k_dim, vd = kv_heads * v_dim;
   const int C = qd + kd + vd;
-  const size_t smem = (size_t)(C + 32) * sizeof(float);
+  const size_t smem = (size_t)(C + 32 + rot_dims) * sizeof(float);
   LLM_HOST_CHECK(smem <= 200 * 1024, ERR_BAD_SIZE);
   const int threads = C >= 2048 ? 512 : (C >= 512 ? 256 : 128);
   PagedCacheKV cache{cache_k, cache_v, block_table, page_stride, table_stride, page_tokens, kv_heads, k_dim, v_dim};
@@ -127,7 +145,7 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
       cudaFuncSetAttribute(conv_norm_cache_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     launch_kernel(conv_norm_cache_kernel<T>, n_tokens, threads, smem, stream, (const T*)u, u_stride, conv_w, taps, \
                   ring, q_norm_w, k_norm_w, (T*)q_out, cache, positions, row_seq, seq_slot, seq_q_start, qd, kd, vd, \
-                  eps, temp_coef, temp_every, write_cache);                                                        \
+                  eps, temp_coef, temp_every, write_cache, inv_freq, rot_dims, halves);                                                        \
   } while (0)
   if (dtype == DT_F32) LAUNCH(float);
   else if (dtype == DT_BF16) LAUNCH(__nv_bfloat16);

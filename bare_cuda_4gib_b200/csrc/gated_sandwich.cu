@@ -2,7 +2,8 @@
 // every sublayer's result, and hands a weighted sum of all earlier layers' results on to the next layer:
 //
 //   y <- y * sigmoid(g + b)            (g the gate's projection of the sublayer's own input, b its bias)
-//   x <- x + rms_norm(y) * p           (p the weight of the norm behind the sublayer)
+//   x <- x + rms_norm(y) * p           (p the weight of the norm behind the sublayer; without that norm
+//                                       x <- x + y * p, p a factor per channel)
 //   X_k <- x;  x <- sum_{j <= k} a[j] X_j      (at a layer's end: X_0 is the embedding's output, X_k layer k - 1's)
 //   h = rms_norm(x) * w                (the next sublayer's input, or the final norm of the wanted rows)
 //
@@ -25,6 +26,7 @@ struct GatedStep {
   long long gate_stride;
   const float* gate_bias;     // [hidden] or null
   const float* post_w;        // [hidden]
+  int post_norm;              // 0: y is only multiplied by post_w
   float post_eps;
   float* history;             // entries `history_stride` elements apart, each [rows, hidden]
   long long history_stride;
@@ -57,7 +59,7 @@ __global__ void __launch_bounds__(GS_THREADS) gated_step_kernel(GatedStep a) {
       row_cache[i] = v;
       sq += v * v;
     }
-    const float s1 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + a.post_eps);
+    const float s1 = a.post_norm ? 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + a.post_eps) : 1.0f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) row_cache[i] = x[i] + row_cache[i] * s1 * a.post_w[i];
   } else {
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) row_cache[i] = x[i];
@@ -141,7 +143,7 @@ __global__ void __launch_bounds__(THREADS) gated_step_vec_kernel(GatedStep a) {
       v[j] = acc;
       sq += acc.x * acc.x + acc.y * acc.y + acc.z * acc.z + acc.w * acc.w;
     }
-    const float s1 = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + a.post_eps);
+    const float s1 = a.post_norm ? 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + a.post_eps) : 1.0f;
 #pragma unroll
     for (int j = 0; j < GS_PIECES; ++j) {
       const int i = threadIdx.x + j * THREADS;
@@ -208,7 +210,7 @@ __global__ void __launch_bounds__(THREADS) gated_step_vec_kernel(GatedStep a) {
 // gate_dtype: element type of the gate's projection; out_dtype: of `out`.
 extern "C" int llm_gated_sandwich_step(float* residual, const float* y, int n_partials, long long partial_stride,
                                        const void* gate, int gate_dtype, long long gate_stride, const float* gate_bias,
-                                       const float* post_w, float post_eps, float* history, long long history_stride,
+                                       const float* post_w, int post_norm, float post_eps, float* history, long long history_stride,
                                        int store_at, const float* mix_w, int mix_n, const float* next_w, float next_eps,
                                        void* out, int out_dtype, const int32_t* row_index, int rows, int hidden,
                                        cudaStream_t stream) {
@@ -218,7 +220,7 @@ extern "C" int llm_gated_sandwich_step(float* residual, const float* y, int n_pa
   LLM_HOST_CHECK((!y || post_w) && (!out || next_w) && (!gate || y), ERR_BAD_SIZE);
   LLM_HOST_CHECK((store_at < 0 && !mix_w) || history, ERR_BAD_SIZE);
   LLM_HOST_CHECK(!mix_w || (mix_n >= 1 && store_at == mix_n - 1), ERR_BAD_SIZE);
-  GatedStep a{residual, y, n_partials, partial_stride, gate, gate_stride, gate_bias, post_w, post_eps, history,
+  GatedStep a{residual, y, n_partials, partial_stride, gate, gate_stride, gate_bias, post_w, post_norm, post_eps, history,
               history_stride, store_at, mix_w, mix_n, next_w, next_eps, out, row_index, hidden};
   // pieces of four where every pointer allows them; few rows: a block of 1,024 threads a row, so that a
   // step of a handful of tokens does not wait on eight dependent loads a thread

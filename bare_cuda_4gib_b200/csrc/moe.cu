@@ -5,7 +5,8 @@
 //   out = sum_k weight_k * W_down,e_k (act(W_gate,e_k h) * (W_up,e_k h)),   act(z) = z * sigmoid(z),
 //
 // plus, where the layer has one, a shared expert that every token uses, times sigmoid(w_sg . h).
-// Router logits, softmax, weights and the shared gate are float32.
+// Router logits, softmax, weights and the shared gate are float32.  Options of the router: a bias per logit, and
+// weights from the softmax over the chosen experts' logits alone (the choice then goes by the logits).
 //
 // Kernels: moe_route (a block per token: logits, softmax, choice, weights, shared gate), moe_sort (one
 // block: tokens' slots grouped by expert, and the list of row tiles the grouped products walk),
@@ -51,7 +52,8 @@ __global__ void __launch_bounds__(MOE_ROUTE_WARPS * 32)
 moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restrict__ w_router,
                  const TW* __restrict__ w_shared_gate, int hidden, int experts, int top, float router_scale,
                  int32_t* __restrict__ ids, float* __restrict__ weights, float* __restrict__ shared_gate, int n_tokens,
-                 const float* __restrict__ correction, int groups, int keep) {
+                 const float* __restrict__ correction, int groups, int keep, const float* __restrict__ bias,
+                 int chosen_softmax) {
   pdl_launch_dependents();
   pdl_wait();
   // a block per token: its warps share the experts' dot products (and the shared gate's, counted as one
@@ -66,22 +68,25 @@ moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restri
     const TW* w = e < experts ? w_router + (long long)e * hidden : w_shared_gate;
     const float dot = warp_sum(lane_dot(x, w, hidden, lane));
     if (lane == 0) {
-      if (e < experts) s[e] = dot;
+      if (e < experts) s[e] = bias ? dot + bias[e] : dot;
       else shared_gate[t] = 1.0f / (1.0f + expf(-dot));
     }
   }
   __syncthreads();
   if (warp != 0) return;
-  float mx = -INFINITY;
-  for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, s[e]);
-  mx = warp_max(mx);
-  float sum = 0.0f;
-  for (int e = lane; e < experts; e += 32) {
-    const float p = expf(s[e] - mx);
-    s[e] = p;
-    sum += p;
+  float sum = 1.0f;
+  if (!chosen_softmax) {      // otherwise the score stays the logit, and the weights are made after the choice
+    float mx = -INFINITY;
+    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, s[e]);
+    mx = warp_max(mx);
+    sum = 0.0f;
+    for (int e = lane; e < experts; e += 32) {
+      const float p = expf(s[e] - mx);
+      s[e] = p;
+      sum += p;
+    }
+    sum = warp_sum(sum);
   }
-  sum = warp_sum(sum);
   __syncwarp();
   // the score is the softmax; the choice goes by score + correction (where the router has one)
   for (int e = lane; e < experts; e += 32) {
@@ -135,15 +140,25 @@ moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restri
       ids[(long long)t * top + k] = at;
       weights[(long long)t * top + k] = s[at] * router_scale;
       choice[at] = -INFINITY;
+      group_best[k] = s[at];      // (the groups' values are no longer needed: the chosen ones' scores in order)
     }
     __syncwarp();
+  }
+  if (chosen_softmax) {
+    float mx = -INFINITY;
+    for (int k = lane; k < top; k += 32) mx = fmaxf(mx, group_best[k]);
+    mx = warp_max(mx);
+    sum = 0.0f;
+    for (int k = lane; k < top; k += 32) sum += expf(group_best[k] - mx);
+    sum = warp_sum(sum);
+    for (int k = lane; k < top; k += 32) weights[(long long)t * top + k] = expf(group_best[k] - mx) / sum * router_scale;
   }
 }
 
 extern "C" int llm_moe_route(const void* h, int dtype, long long h_stride, const void* w_router, const void* w_shared_gate,
                              int w_dtype, int hidden, int experts, int top, float router_scale, int32_t* ids,
                              float* weights, float* shared_gate, int n_tokens, const float* correction, int groups,
-                             int keep, cudaStream_t stream) {
+                             int keep, const float* bias, int chosen_softmax, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   LLM_HOST_CHECK(experts >= 1 && experts <= MOE_MAX_EXPERTS && top >= 1 && top <= experts, ERR_BAD_SIZE);
   LLM_HOST_CHECK(groups <= 1 || (experts % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (experts / groups)),
@@ -152,7 +167,7 @@ extern "C" int llm_moe_route(const void* h, int dtype, long long h_stride, const
 #define ROUTE(T, TW)                                                                                                 \
   launch_kernel(moe_route_kernel<T, TW>, blocks, MOE_ROUTE_WARPS * 32, 0, stream, (const T*)h, h_stride,              \
                 (const TW*)w_router, (const TW*)w_shared_gate, hidden, experts, top, router_scale, ids, weights,        \
-                shared_gate, n_tokens, correction, groups, keep)
+                shared_gate, n_tokens, correction, groups, keep, bias, chosen_softmax)
   if (dtype == DT_F32 && w_dtype == DT_F32) ROUTE(float, float);
   else if (dtype == DT_BF16 && w_dtype == DT_BF16) ROUTE(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == DT_BF16 && w_dtype == DT_F32) ROUTE(__nv_bfloat16, float);

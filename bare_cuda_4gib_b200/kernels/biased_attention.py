@@ -21,7 +21,7 @@ def lib():
         l = build.load_library("biased_attention.cu")
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
         l.llm_conv_norm_cache.argtypes = [P, I, L, P, I, P, P, P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, I, I, F, F,
-                                          I, I, P]
+                                          I, I, P, I, I, P]
         l.llm_conv_ring_write.argtypes = [P, I, L, P, I, I, P, P, P, P, I, P]
         l.llm_biased_attention.argtypes = [P, P, I, L, P, P, P, L, I, I, I, I, I, P, I, P, P, I, I, F, I, F, F, I, P, P, L, P]
         for name in ("llm_conv_norm_cache", "llm_conv_ring_write", "llm_biased_attention"):
@@ -32,18 +32,20 @@ def lib():
 
 def conv_norm_cache(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, q_norm_w: torch.Tensor,
                     k_norm_w: torch.Tensor, q_out: torch.Tensor, cache: CacheView, q_heads: int, eps: float,
-                    temp_coef: float, temp_every: int, write_cache: bool) -> None:
+                    temp_coef: float, temp_every: int, write_cache: bool, inv_freq: Optional[torch.Tensor] = None,
+                    rot_dims: int = 0, halves: bool = False) -> None:
     """u [rows, q | k | v channels] (may be a column view) -> causal convolution over time with
     `conv_w` [channels, taps] (history before the step from `ring`), RMS norm of all q channels and
-    of all k channels, the position factor on q; q to `q_out`, k and v into the cache."""
-    _dev(u, conv_w, ring, q_norm_w, k_norm_w, q_out)
+    of all k channels, the position factor on q; with `inv_freq` the first `rot_dims` entries of every q and
+    k head turned by position (neighbouring pairs, or `halves`); q to `q_out`, k and v into the cache."""
+    _dev(u, conv_w, ring, q_norm_w, k_norm_w, q_out, inv_freq)
     _check(lib().llm_conv_norm_cache(
         u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(),
         q_norm_w.data_ptr(), k_norm_w.data_ptr(), q_out.data_ptr(), cache.k_ptr, cache.v_ptr,
         cache.block_table.data_ptr(), cache.page_stride, cache.table_stride, cache.page_tokens, cache.kv_heads,
         cache.head_dim, cache.v_dim, ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
         ctx.seq_q_start.data_ptr(), ctx.n_tokens, q_heads, float(eps), float(temp_coef), int(temp_every),
-        1 if write_cache else 0, ctx.stream), "conv_norm_cache")
+        1 if write_cache else 0, _ptr(inv_freq), int(rot_dims), 1 if halves else 0, ctx.stream), "conv_norm_cache")
 
 
 def conv_ring_write(ctx, u: torch.Tensor, ring: torch.Tensor, taps: int, channels: int) -> None:

@@ -1,0 +1,105 @@
+"""Launchers of `csrc/gated_delta.cu` and `csrc/gated_delta_chunked.cu`: the gated delta rule over a step's
+tokens (operands, scan, chunks on the tensor cores) and in one kernel for steps of one token per request."""
+
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_longlong, c_void_p
+from typing import Optional
+
+import torch
+
+from . import build
+from .lib import _check, _dev, dtype_code
+
+MAX_KEY_DIM = 1024
+STEP_MAX_SHARED = 160 * 1024
+_lib = None
+
+
+def lib():
+    global _lib
+    if _lib is None:
+        l = build.load_library("gated_delta.cu")
+        P, I, L, F = c_void_p, c_int, c_longlong, c_float
+        l.llm_gated_delta_operands.argtypes = [P, I, L, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, F, F, P]
+        l.llm_gated_delta_scan.argtypes = [P, P, P, P, L, I, P, L, I, P, P, I, P, P, P, P, P, I, I, I, I, I, P]
+        l.llm_gated_delta_step.argtypes = [P, I, L, P, I, P, P, L, I, P, L, I, P, P, I, P, P, L, I, I, P, P, L, P, P, P, I, I, I,
+                                           I, I, I, F, F, F, P]
+        l.llm_gated_delta_step_shared_bytes.argtypes = [I, I]
+        l.llm_gated_delta_step_shared_bytes.restype = c_longlong
+        for name in ("llm_gated_delta_operands", "llm_gated_delta_scan", "llm_gated_delta_step"):
+            getattr(l, name).restype = c_int
+        _lib = l
+    return _lib
+
+
+class Gates:
+    """Where a token's decays and step size come from: `z` [rows, heads] or (with `channel`) [rows, heads * dim]
+    and `b` [rows, heads], pre-activations that may be column views; `a_log` [heads], `dt_bias` like z's
+    columns, float32.  decay = exp(-exp(a_log) softplus(z + dt_bias)), step size = sigmoid(b)."""
+
+    __slots__ = ("z", "b", "a_log", "dt_bias", "channel")
+
+    def __init__(self, z: torch.Tensor, b: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, channel: bool):
+        _dev(z, b, a_log, dt_bias)
+        if z.stride(-1) != 1 or b.stride(-1) != 1 or a_log.dtype != torch.float32 or dt_bias.dtype != torch.float32:
+            raise TypeError("gated delta: gates not as the kernels need")
+        self.z, self.b, self.a_log, self.dt_bias, self.channel = z, b, a_log, dt_bias, channel
+
+    def arguments(self):
+        return (self.z.data_ptr(), self.z.stride(0), dtype_code(self.z.dtype), self.b.data_ptr(), self.b.stride(0),
+                dtype_code(self.b.dtype), self.a_log.data_ptr(), self.dt_bias.data_ptr(), 1 if self.channel else 0)
+
+
+def _floats(what: str, *tensors: Optional[torch.Tensor]) -> None:
+    _dev(*tensors)
+    for t in tensors:
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise TypeError(f"gated delta {what}: constants, states and operands must be contiguous float32")
+
+
+def operands(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, qn: torch.Tensor, kn: torch.Tensor,
+             vn: torch.Tensor, kv_heads: int, dk: int, heads: int, dv: int, unit_eps: float) -> None:
+    """u [rows, q | k | v | ...]: the convolution (history before the step from `ring`) and silu; qn, kn [rows,
+    kv_heads * dk] the unit vectors (q also / sqrt(dk)), vn [rows, heads * dv].  All float32."""
+    _floats("operands", conv_w, ring, qn, kn, vn)
+    _check(lib().llm_gated_delta_operands(
+        u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(), qn.data_ptr(),
+        kn.data_ptr(), vn.data_ptr(), ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
+        ctx.seq_q_start.data_ptr(), ctx.n_tokens, kv_heads, dk, heads, dv, float(unit_eps), dk ** -0.5, ctx.stream),
+        "gated_delta_operands")
+
+
+def scan(ctx, qn: torch.Tensor, kn: torch.Tensor, vn: torch.Tensor, gates: Gates, state: torch.Tensor, out: torch.Tensor,
+         heads: int, kv_heads: int, dk: int, dv: int) -> None:
+    """Every request's new tokens in order: S = g S; u = beta (v - S^T k); S += k u^T; out = S^T q, with S in
+    `state[slot]` ([heads, dk, dv] float32) read at the start and left at the end.  out [rows, heads * dv]."""
+    _floats("scan", qn, kn, vn, state, out)
+    _check(lib().llm_gated_delta_scan(
+        qn.data_ptr(), kn.data_ptr(), vn.data_ptr(), *gates.arguments(), state.data_ptr(), out.data_ptr(),
+        ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.seq_q_len.data_ptr(), ctx.n_seqs, heads, kv_heads, dk, dv,
+        ctx.stream), "gated_delta_scan")
+
+
+def step_takes(dk: int, dv: int) -> bool:
+    """Whether the kernel for steps of one token per request takes these head sizes."""
+    need = int(lib().llm_gated_delta_step_shared_bytes(dk, dv))
+    return 0 < need <= STEP_MAX_SHARED
+
+
+def step(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, gates: Gates, state: torch.Tensor,
+         gate: torch.Tensor, gate_kind: str, norm_w: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dk: int,
+         dv: int, unit_eps: float, eps: float, write_ring: bool) -> None:
+    """A step of one token per request, a block per (request, head): everything from the stored projections to
+    what the output projection reads.  `gate` [rows, heads * dv] pre-activations of `gate_kind` ("silu" or
+    "sigmoid"), possibly a column view; out [rows, heads * dv] = rms_norm per head * norm_w * gate."""
+    _floats("step", conv_w, ring, state, norm_w)
+    _dev(u, gate, out)
+    if out.dtype != u.dtype or gate.stride(1) != 1:
+        raise TypeError("gated delta step: element types or layout not as the kernel needs")
+    _check(lib().llm_gated_delta_step(
+        u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(),
+        *gates.arguments(), state.data_ptr(), gate.data_ptr(), gate.stride(0), dtype_code(gate.dtype),
+        {"silu": 1, "sigmoid": 0}[gate_kind], norm_w.data_ptr(), out.data_ptr(), out.stride(0), ctx.positions.data_ptr(),
+        ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.n_seqs, heads, kv_heads, dk, dv, 1 if write_ring else 0,
+        float(unit_eps), dk ** -0.5, float(eps), ctx.stream), "gated_delta_step")

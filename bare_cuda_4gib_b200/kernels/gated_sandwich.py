@@ -20,7 +20,7 @@ def lib():
     if _lib is None:
         l = build.load_library("gated_sandwich.cu")
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
-        l.llm_gated_sandwich_step.argtypes = [P, P, I, L, P, I, L, P, P, F, P, L, I, P, I, P, F, P, I, P, I, I, P]
+        l.llm_gated_sandwich_step.argtypes = [P, P, I, L, P, I, L, P, P, I, F, P, L, I, P, I, P, F, P, I, P, I, I, P]
         l.llm_gated_sandwich_step.restype = c_int
         _lib = l
     return _lib
@@ -39,13 +39,14 @@ class DepthMix:
 
 class GatedDelta:
     """A sublayer's result `y` that still has to be gated (`gate` pre-activations [rows, width] with
-    `gate_bias`, or None), normed (`weight` float32, `eps`) and added to the stream, and what happens to
-    the stream right after (`depth`, or None).  With `y` None only `depth` applies."""
+    `gate_bias`, or None), normed (`weight` float32, `eps`; with `eps` None only multiplied by `weight`) and
+    added to the stream, and what happens to the stream right after (`depth`, or None).  With `y` None only
+    `depth` applies."""
 
     __slots__ = ("y", "gate", "gate_bias", "weight", "eps", "depth")
 
     def __init__(self, y: Optional[Partials], gate: Optional[torch.Tensor], gate_bias: Optional[torch.Tensor],
-                 weight: Optional[torch.Tensor], eps: float, depth: Optional[DepthMix] = None):
+                 weight: Optional[torch.Tensor], eps: Optional[float], depth: Optional[DepthMix] = None):
         self.y, self.gate, self.gate_bias, self.weight, self.eps, self.depth = y, gate, gate_bias, weight, eps, depth
 
 
@@ -67,7 +68,8 @@ def step(residual: torch.Tensor, delta: Optional[GatedDelta], weight: Optional[t
         residual.data_ptr(), _ptr(y.tensor) if y is not None else 0, y.n if y is not None else 0,
         y.stride if y is not None else 0, _ptr(gate), dtype_code(gate.dtype) if gate is not None else 0,
         gate.stride(0) if gate is not None else 0, _ptr(delta.gate_bias) if y is not None else 0,
-        _ptr(delta.weight) if y is not None else 0, float(delta.eps) if y is not None else 0.0,
+        _ptr(delta.weight) if y is not None else 0, 0 if y is not None and delta.eps is None else 1,
+        float(delta.eps) if y is not None and delta.eps is not None else 0.0,
         _ptr(hist), hist.stride(0) if hist is not None else 0, depth.index if depth is not None else -1,
         _ptr(depth.weights) if depth is not None else 0, depth.index + 1 if depth is not None else 0,
         _ptr(weight), float(eps), _ptr(out), dtype_code(out.dtype) if out is not None else 0, _ptr(row_index), rows,

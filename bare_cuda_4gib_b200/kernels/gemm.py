@@ -94,7 +94,8 @@ class GemmPlan:
         if m is None:
             esize = a.element_size()
             storage_left = a.untyped_storage().nbytes() - a.storage_offset() * esize
-            capacity = max(a.shape[0], storage_left // (a.stride(0) * esize))
+            # rows that lie wholly inside the storage (`a` may be a column view, whose last row ends early)
+            capacity = max(a.shape[0], (storage_left // esize - self.k) // a.stride(0) + 1)
             m = tensor_map(a.data_ptr(), capacity, self.k, a.stride(0), bn)
             self.act_maps[key] = m
         return m

@@ -20,7 +20,7 @@ def lib():
     if _lib is None:
         l = build.load_library("moe.cu")
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
-        l.llm_moe_route.argtypes = [P, I, L, P, P, I, I, I, I, F, P, P, P, I, P, I, I, P]
+        l.llm_moe_route.argtypes = [P, I, L, P, P, I, I, I, I, F, P, P, P, I, P, I, I, P, I, P]
         l.llm_moe_sort.argtypes = [P, I, I, I, P, P, P, P]
         l.llm_moe_grouped.argtypes = [P, L, P, P, I, I, P, P, P, P, I, I, I, I, I, P]
         l.llm_moe_combine.argtypes = [P, I, P, I, I, L, P, P, I, I, P, P, I, P, I, L, P]
@@ -49,13 +49,18 @@ def max_tiles(n_slots: int, experts: int, tensor_cores: bool = False) -> int:
 
 def route(ctx, h: torch.Tensor, w_router: torch.Tensor, w_shared_gate: Optional[torch.Tensor], top: int,
           router_scale: float, ids: torch.Tensor, weights: torch.Tensor, shared_gate: Optional[torch.Tensor], rows: int,
-          correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1) -> None:
+          correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, bias: Optional[torch.Tensor] = None,
+          chosen_softmax: bool = False) -> None:
     """ids, weights [rows, top]: the `top` experts with the largest softmax(W_router h) (float32), and
     that score times `router_scale`; shared_gate [rows] = sigmoid(w_shared_gate . h).  With `correction`
     (float32, one per expert) the choice goes by score + correction while the weight stays the score; with
     `groups` > 1 the experts form that many equal groups of neighbours and only experts of the `keep`
-    groups with the largest best choice value can be chosen."""
-    _dev(h, w_router, w_shared_gate, ids, weights, shared_gate, correction)
+    groups with the largest best choice value can be chosen.  `bias` (float32, one per expert) is added to the
+    logits; with `chosen_softmax` the choice goes by the logits and the weights are the softmax over the chosen
+    experts' logits only, times `router_scale`."""
+    _dev(h, w_router, w_shared_gate, ids, weights, shared_gate, correction, bias)
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != w_router.shape[0]):
+        raise TypeError("moe route: the bias must be float32, one number per router output")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != w_router.shape[0]):
         raise TypeError("moe route: the correction must be float32, one number per router output")
     if w_shared_gate is not None and w_shared_gate.dtype != w_router.dtype:
@@ -63,7 +68,7 @@ def route(ctx, h: torch.Tensor, w_router: torch.Tensor, w_shared_gate: Optional[
     _check(lib().llm_moe_route(h.data_ptr(), dtype_code(h.dtype), h.stride(0), w_router.data_ptr(), _ptr(w_shared_gate),
                                dtype_code(w_router.dtype), h.shape[1], w_router.shape[0], top, float(router_scale),
                                ids.data_ptr(), weights.data_ptr(), _ptr(shared_gate), rows, _ptr(correction), int(groups),
-                               int(keep), ctx.stream), "moe_route")
+                               int(keep), _ptr(bias), 1 if chosen_softmax else 0, ctx.stream), "moe_route")
 
 
 def sort(ctx, ids: torch.Tensor, n_slots: int, experts: int, sorted_slots: torch.Tensor, tiles: torch.Tensor,

@@ -19,7 +19,7 @@ import torch
 
 from ..errors import ConfigError
 from ..kernels import lib as K
-from .base import KVCacheRequest, Part
+from .base import KVCacheRequest, Part, StateRequest
 from .linear import Linear
 from .registry import build_part, register_mixer
 from ..weights.loader import fused_rows
@@ -217,7 +217,11 @@ class GeneralAttention(Part):
     mean square per head after the rotation (`unit_qk`, without weights); blocks of positions (`chunk`: a
     query sees its own block only, blocks counted from position 0); a learned number per head whose
     exponential joins the softmax's denominator (`sink`); and one sigmoid gate per head on its output,
-    read from the mixer's input (`head_gate`).
+    read from the mixer's input (`head_gate`); a short causal convolution over time on every channel of q, k
+    and v ahead of norm and rotation (`taps`: its length; the last taps - 1 projected rows of a request are its
+    state); `qk_norm` "all", one RMS norm over all heads of q and one over all heads of k, with a weight per
+    channel (with `taps`); and a constant in the place of the learned sink (`sink_score`: 0 adds one to the
+    denominator).
 
     One product makes [q | k | v (| g)]; one kernel adds the biases, norms, turns, mixes and caches; then the
     engine's tensor-core attention kernels run in bfloat16 steps (all three for equal key and value sizes
@@ -225,11 +229,12 @@ class GeneralAttention(Part):
     float32 steps and for sizes that are no multiples of 16 up to 128.  All of them join the sink and apply
     the gate where they finish a row.
 
-    params: `hidden`, `heads`, `kv_heads`, `dim`, `vdim`, `scale`, `eps`, `bias` (bool), `qk_norm` (bool),
-    `unit_qk` (bool), `softcap` (None: no cap), `window`, `chunk` (None: every key), `sink` (bool), `head_gate`
-    (bool), `v_mix` (None | "source" | "mix"), `position`.
-    tensors: `q`, `k`, `v`, `o`, (`q_bias`, `k_bias`, `v_bias`,) (`q_norm`, `k_norm` [dim],) (`v_lambda` [],)
-    (`sink` [heads],) (`g` [heads, hidden])."""
+    params: `hidden`, `heads`, `kv_heads`, `dim`, `vdim`, `scale`, `eps`, `bias` (bool), `qk_norm` (bool or
+    "all"), `unit_qk` (bool), `softcap` (None: no cap), `window`, `chunk` (None: every key), `sink` (bool),
+    `sink_score` (None: no constant), `head_gate` (bool), `v_mix` (None | "source" | "mix"), `taps` (None: no
+    convolution), `position`.
+    tensors: `q`, `k`, `v`, `o`, (`q_bias`, `k_bias`, `v_bias`,) (`q_norm`, `k_norm` [dim], or [channels] for
+    "all",) (`q_conv`, `k_conv`, `v_conv` [channels, taps],) (`v_lambda` [],) (`sink` [heads],) (`g` [heads, hidden])."""
 
     takes_lazy_input = False
 
@@ -248,6 +253,14 @@ class GeneralAttention(Part):
         if self.qk_norm and self.unit_qk:
             raise ConfigError("general_attention: queries and keys are normed with weights or without, not both")
         self.has_sink, self.head_gate = bool(p.get("sink")), bool(p.get("head_gate"))
+        self.sink_score = p.get("sink_score")
+        if self.has_sink and self.sink_score is not None:
+            raise ConfigError("general_attention: the sink is learned or a constant, not both")
+        self.norm_all, self.taps = p.get("qk_norm") == "all", int(p.get("taps") or 0)
+        # the kernel with the convolution norms over all heads and has none of the other steps ahead of the scores
+        if self.norm_all != (self.taps > 0) or (self.taps and (self.has_bias or self.unit_qk or p.get("v_mix"))):
+            raise ConfigError("general_attention: a convolution (`taps`) goes with qk_norm 'all' and without biases, "
+                              "unit_qk and v_mix")
         self.softcap = float(p["softcap"]) if p.get("softcap") else 0.0
         self.v_mix = p.get("v_mix")
         if self.v_mix not in (None, "source", "mix"):
@@ -266,7 +279,11 @@ class GeneralAttention(Part):
         if self.has_bias:
             out.update({"q_bias": ((self.qd,), "zero"), "k_bias": ((self.kd,), "zero"), "v_bias": ((self.vd,), "zero")})
         if self.qk_norm:
-            out.update({"q_norm": ((self.dim,), "norm"), "k_norm": ((self.dim,), "norm")})
+            out.update({"q_norm": ((self.qd if self.norm_all else self.dim,), "norm"),
+                        "k_norm": ((self.kd if self.norm_all else self.dim,), "norm")})
+        if self.taps:
+            out.update({"q_conv": ((self.qd, self.taps), "unit"), "k_conv": ((self.kd, self.taps), "unit"),
+                        "v_conv": ((self.vd, self.taps), "unit")})
         if self.v_mix is not None:
             out["v_lambda"] = ((), "zero")      # the source layer has the tensor too and does not use it
         if self.has_sink:
@@ -290,7 +307,9 @@ class GeneralAttention(Part):
         return KVCacheRequest(self.kv_heads, self.dim, self._span(), None if self.vdim == self.dim else self.vdim)
 
     def state_request(self):
-        return None
+        if not self.taps:
+            return None
+        return StateRequest((max(self.taps - 1, 1), self.qd + self.kd + self.vd), torch.float32)
 
     def prepare(self, dtype, device) -> None:
         t = self.tensors
@@ -300,8 +319,11 @@ class GeneralAttention(Part):
         self.o.prepare(dtype)
         self.bias = (torch.cat([t[n].to(torch.float32).reshape(-1) for n in ("q_bias", "k_bias", "v_bias")]).contiguous()
                      if self.has_bias else None)
-        self.q_norm = t["q_norm"].to(dtype).contiguous() if self.qk_norm else None
-        self.k_norm = t["k_norm"].to(dtype).contiguous() if self.qk_norm else None
+        norm_dtype = torch.float32 if self.norm_all else dtype
+        self.q_norm = t["q_norm"].to(norm_dtype).contiguous() if self.qk_norm else None
+        self.k_norm = t["k_norm"].to(norm_dtype).contiguous() if self.qk_norm else None
+        self.conv_w = (torch.cat([t[n] for n in ("q_conv", "k_conv", "v_conv")], 0).to(torch.float32).contiguous()
+                       if self.taps else None)
         self.v_lambda = float(t["v_lambda"].to(torch.float32).reshape(-1)[0].item()) if self.v_mix == "mix" else 0.0
         self.position.prepare(dtype, device)
         self.inv_freq = getattr(self.position, "inv_freq", None)
@@ -312,7 +334,11 @@ class GeneralAttention(Part):
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         if self.unit_qk and self.magnitude != 1.0:
             raise ConfigError("general_attention: queries and keys of unit size take a rotation that keeps their size")
+        if self.taps and self.magnitude != 1.0:
+            raise ConfigError("general_attention: the kernel with the convolution takes a rotation that keeps the heads' size")
         self.sink = t["sink"].to(torch.float32).contiguous() if self.has_sink else None
+        if self.sink_score is not None:
+            self.sink = torch.full((self.heads,), float(self.sink_score), dtype=torch.float32, device=device)
         self.fast = None
         if dtype == torch.bfloat16 and device.type == "cuda":
             # equal head sizes without a cap: the engine's tcgen05 prefill, cluster decode and mma.sync kernels;
@@ -326,16 +352,18 @@ class GeneralAttention(Part):
             fast.step_tiles(ctx, self.fast)
 
     def forward(self, ctx, call, h):
-        from ..kernels import biased_attention as BA, head_prepare as HP
+        from ..kernels import biased_attention as BA
         n = ctx.n_tokens
         u = self.proj.forward(ctx, h, n, ctx.dtype, "mixer_in").tensor
         q = ctx.ws.get("q", (n, self.qd), ctx.dtype)
         shared = ctx.ws.get("mixed_values", (n, self.vd), torch.float32) if self.v_mix else None
-        HP.headnorm_rope_cache(ctx, u, 0, self.qd, self.qd + self.kd, self.q_norm, self.k_norm, self.eps, self.inv_freq,
-                               self.rot_dims, self.magnitude, q, call.cache, self.heads, call.writes_cache,
-                               halves=self.halves, bias=self.bias, v_mix_in=shared if self.v_mix == "mix" else None,
-                               v_mix=self.v_lambda, v_mix_out=shared if self.v_mix == "source" else None,
-                               unit_norm=self.unit_qk)
+        if self.taps:
+            BA.conv_norm_cache(ctx, u, self.conv_w, call.state, self.q_norm, self.k_norm, q, call.cache, self.heads, self.eps,
+                               0.0, 1, call.writes_cache, self.inv_freq, self.rot_dims, self.halves)
+            if call.writes_cache:
+                BA.conv_ring_write(ctx, u, call.state, self.taps, self.qd + self.kd + self.vd)
+        else:
+            self._prepare_heads(ctx, call, u, q, shared)
         out = ctx.ws.get("attn_out", (n, self.heads * self.vdim), ctx.dtype)
         window = int(self.window) if self.window else 0
         extras = K.AttentionExtras(self.chunk or 0, self.sink, u[:, u.shape[1] - self.heads:] if self.head_gate else None)
@@ -345,3 +373,11 @@ class GeneralAttention(Part):
         else:
             BA.attention(ctx, q, out, call.cache, None, self.heads, self.scale, window, 1.0, self.softcap, extras)
         return self.o.forward(ctx, out, n, torch.float32, "attn_proj", allow_partials=True)
+
+    def _prepare_heads(self, ctx, call, u, q, shared) -> None:
+        from ..kernels import head_prepare as HP
+        HP.headnorm_rope_cache(ctx, u, 0, self.qd, self.qd + self.kd, self.q_norm, self.k_norm, self.eps, self.inv_freq,
+                               self.rot_dims, self.magnitude, q, call.cache, self.heads, call.writes_cache,
+                               halves=self.halves, bias=self.bias, v_mix_in=shared if self.v_mix == "mix" else None,
+                               v_mix=self.v_lambda, v_mix_out=shared if self.v_mix == "source" else None,
+                               unit_norm=self.unit_qk)

@@ -88,3 +88,46 @@ class SandwichBlock:
             h = self.ffn_norm.forward(ctx, residual, pending, n)
             pending = self.post2.pending(self.ffn.forward(ctx, h))
         return pending
+
+
+@register_block("scaled_prenorm")
+class ScaledPreNormBlock:
+    """x += s1 * mixer(norm(x)), then (if the layer has a feed-forward) x += s2 * ff(norm(x)), s1 and s2 one
+    factor per channel: `layer_spec.extras["scale1"]` and `["scale2"]` (norm parts that lend a `factor`).  A
+    sublayer's result is handed on unscaled and un-added; the norm that reads the stream next
+    (`gated_sandwich_rmsnorm`) does both first, in its own kernel."""
+
+    def __init__(self, layer_spec):
+        self.mixer_norm = build_part("norm", layer_spec.mixer_norm)
+        self.mixer = build_part("mixer", layer_spec.mixer)
+        self.scale1 = build_part("norm", layer_spec.extras["scale1"])
+        self.has_ffn = layer_spec.ffn is not None
+        if self.has_ffn:
+            self.ffn_norm = build_part("norm", layer_spec.ffn_norm)
+            self.ffn = build_part("feed_forward", layer_spec.ffn)
+            self.scale2 = build_part("norm", layer_spec.extras["scale2"])
+
+    def parts(self):
+        out = [self.mixer_norm, self.mixer, self.scale1]
+        if self.has_ffn:
+            out += [self.ffn_norm, self.ffn, self.scale2]
+        return out
+
+    def cache_demands(self):
+        many = getattr(self.mixer, "cache_demands", None)
+        return many() if many else [(self.mixer.cache_request(), self.mixer.state_request())]
+
+    def entry_norm(self):
+        return self.mixer_norm
+
+    def forward(self, ctx, call, residual, pending):
+        from ..kernels.gated_sandwich import GatedDelta
+        n = ctx.n_tokens
+        ctx.residual = None          # sublayers hand their result back: it is scaled before it is added
+        ctx.following_norm = None
+        h = self.mixer_norm.forward(ctx, residual, pending, n)
+        pending = GatedDelta(self.mixer.forward(ctx, call, h), None, None, self.scale1.factor, None)
+        if self.has_ffn:
+            h = self.ffn_norm.forward(ctx, residual, pending, n)
+            pending = GatedDelta(self.ffn.forward(ctx, h), None, None, self.scale2.factor, None)
+        return pending

@@ -21,15 +21,19 @@ Options beside that form (each off unless its parameter is given):
   whose result is h itself (times the weight);
 * `correction`: a tensor with one number per router output that is added to the score for the choice
   only; the weight stays the score;
+* `router_bias`: a tensor with one number per router output that is added to its logit;
+* `weights` "chosen": the choice goes by the logits and a token's weights are the softmax over its chosen
+  experts' logits only (times `router_scale`);
 * `groups`, `keep`: the router's outputs (identity experts included) form `groups` equal groups of
   neighbours, a group counts by its largest choice value, and only experts of the `keep` best groups can
   be chosen.
 
 params: `hidden`, `experts`, `top`, `router_scale`, `intermediate`, `shared_intermediate` (None: no shared
-expert), `shared_gate` (bool), `expert_form`, `identity`, `correction` (bool), `groups`, `keep`.
-tensors: `router` [experts + identity, hidden], `correction` [experts + identity], `e<j>.gate|up`
-[intermediate, hidden] (relu2: `e<j>.up` only), `e<j>.down` [hidden, intermediate], `shared.gate|up|down`,
-`shared.sg` [1, hidden].
+expert), `shared_gate` (bool), `expert_form` (the shared expert's too), `identity`, `correction` (bool), `groups`,
+`keep`, `router_bias` (bool), `weights` ("all" | "chosen").
+tensors: `router` [experts + identity, hidden], `router_bias`, `correction` [experts + identity], `e<j>.gate|up`
+[intermediate, hidden] (relu2: `e<j>.up` only), `e<j>.down` [hidden, intermediate], `shared.gate|up|down`
+(relu2: without the gate), `shared.sg` [1, hidden].
 """
 
 from __future__ import annotations
@@ -61,6 +65,9 @@ class MixtureOfExperts(Part):
         self.identity = int(p.get("identity") or 0)
         self.outputs = self.experts + self.identity          # what the router scores
         self.has_correction = bool(p.get("correction"))
+        self.has_bias, self.chosen = bool(p.get("router_bias")), p.get("weights", "all") == "chosen"
+        if p.get("weights", "all") not in ("all", "chosen"):
+            raise ConfigError(f"moe: weights '{p.get('weights')}' is not one of ['all', 'chosen']")
         self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or p.get("groups") or 1)
         from ..kernels.moe import MAX_EXPERTS
         if not (1 <= self.top <= self.outputs <= MAX_EXPERTS) or self.experts < 1:
@@ -77,13 +84,15 @@ class MixtureOfExperts(Part):
         out = {"router": ((self.outputs, self.hidden), "matrix")}
         if self.has_correction:
             out["correction"] = ((self.outputs,), "zero")
+        if self.has_bias:
+            out["router_bias"] = ((self.outputs,), "zero")
         for e in range(self.experts):
             for n in self._matrices():
                 out[f"e{e}.{n}"] = ((self.ff, self.hidden), "matrix")
             out[f"e{e}.down"] = ((self.hidden, self.ff), "matrix")
         if self.shared_ff:
-            out["shared.gate"] = ((self.shared_ff, self.hidden), "matrix")
-            out["shared.up"] = ((self.shared_ff, self.hidden), "matrix")
+            for n in self._matrices():
+                out["shared." + n] = ((self.shared_ff, self.hidden), "matrix")
             out["shared.down"] = ((self.hidden, self.shared_ff), "matrix")
             if self.has_shared_gate:
                 out["shared.sg"] = ((1, self.hidden), "matrix")
@@ -92,7 +101,7 @@ class MixtureOfExperts(Part):
     def adjacent_weights(self):
         groups = [tuple(f"e{e}.{t}" for e in range(self.experts) for t in self._matrices()),
                   tuple(f"e{e}.down" for e in range(self.experts))]
-        if self.shared_ff:
+        if self.shared_ff and self.gated:
             groups.append(("shared.gate", "shared.up"))
         return groups
 
@@ -101,13 +110,14 @@ class MixtureOfExperts(Part):
         E = self.experts
         self.w_up = fused_rows([t[f"e{e}.{n}"] for e in range(E) for n in self._matrices()]).to(dtype).contiguous()
         self.correction = t["correction"].to(torch.float32).contiguous() if self.has_correction else None
+        self.router_bias = t["router_bias"].to(torch.float32).contiguous() if self.has_bias else None
         self.w_down = fused_rows([t[f"e{e}.down"] for e in range(E)]).to(dtype).contiguous()
         self.w_router = t["router"].contiguous()
         self.w_sg = t["shared.sg"].to(self.w_router.dtype).reshape(-1).contiguous() if self.has_shared_gate else None
         if self.shared_ff:
-            self.shared_gate_up = Linear(fused_rows([t["shared.gate"], t["shared.up"]]), "moe.shared.gate_up")
+            self.shared_up = Linear(fused_rows([t["shared." + n] for n in self._matrices()]), "moe.shared.up")
             self.shared_down = Linear(t["shared.down"], "moe.shared.down")
-            self.shared_gate_up.prepare(dtype)
+            self.shared_up.prepare(dtype)
             self.shared_down.prepare(dtype)
         from ..kernels.moe import GroupedPlan
         # bfloat16 experts whose rows the copy engine can fetch run on the tensor cores
@@ -132,7 +142,7 @@ class MixtureOfExperts(Part):
         tc = self.plan is not None and ctx.dtype == torch.bfloat16 and h.dtype == torch.bfloat16
         n_tiles = tiles.view(-1)[3 * M.max_tiles(slots, E, tc):]
         M.route(ctx, h, self.w_router, self.w_sg, top, self.router_scale, ids, weights, gate, n, self.correction,
-                self.groups, self.keep)
+                self.groups, self.keep, self.router_bias, self.chosen)
         M.sort(ctx, ids, slots, E, sorted_slots, tiles, n_tiles, tc)
         act = ctx.ws.get("moe_act", (n, top * self.ff), ctx.dtype)
         act_rows = act.view(-1)[: slots * self.ff].view(slots, self.ff)
@@ -152,8 +162,14 @@ class MixtureOfExperts(Part):
                       slots, E)
         shared = None
         if self.shared_ff:
-            a = self.shared_gate_up.forward(ctx, h, n, ctx.dtype, "moe_shared_act", glu="silu")
-            shared = self.shared_down.forward(ctx, a.tensor, n, f32, "moe_shared_out", allow_partials=True)
+            if self.gated:
+                a = self.shared_up.forward(ctx, h, n, ctx.dtype, "moe_shared_act", glu="silu").tensor
+            else:
+                from ..kernels import streams as SK
+                z = self.shared_up.forward(ctx, h, n, ctx.dtype, "moe_shared_up")
+                a = ctx.ws.get("moe_shared_act", (n, self.shared_ff), ctx.dtype)
+                SK.activation(z, a, n, "relu2", ctx.stream)
+            shared = self.shared_down.forward(ctx, a, n, f32, "moe_shared_out", allow_partials=True)
         out = ctx.ws.get("ffn_out", (n, self.hidden), f32)
         if self.identity:
             M.combine(ctx, y, top, shared, gate, out, n, self.hidden, ids, weights, E, h)

@@ -110,15 +110,15 @@ class GatedSandwichRMSNorm(Part):
     weighted sum over the layers so far), in the same kernel; as the norm behind a sublayer it only
     lends its factor (`factor`).
 
-    params: `size`, `eps`, `one_plus` (the weight is stored around zero and the factor is 1 + w).
-    tensors: `weight` [size]."""
+    params: `size`, `eps`, `one_plus` (the weight is stored around zero and the factor is 1 + w), `mult`
+    (optional: a constant that multiplies the factor).  tensors: `weight` [size]."""
 
     def local_weights(self):
         return {"weight": ((self.params["size"],), "zero" if self.params.get("one_plus") else "norm")}
 
     def prepare(self, dtype, device) -> None:
         w = self.tensors["weight"].to(torch.float32)
-        self.factor = ((1.0 + w) if self.params.get("one_plus") else w).contiguous()
+        self.factor = (((1.0 + w) if self.params.get("one_plus") else w) * float(self.params.get("mult", 1.0))).contiguous()
 
     def forward(self, ctx, residual: torch.Tensor, delta, rows: int, row_index: Optional[torch.Tensor] = None,
                 buffer: str = "normed", lazy: bool = False):
@@ -126,3 +126,17 @@ class GatedSandwichRMSNorm(Part):
         out = ctx.ws.get(buffer, (rows, self.params["size"]), ctx.dtype)
         GS.step(residual, delta, self.factor, out, float(self.params["eps"]), rows, row_index, ctx.stream)
         return out
+
+
+@register_norm("layer_scale")
+class LayerScale(Part):
+    """A learned factor per channel on a sublayer's result; as `GatedSandwichRMSNorm` behind a sublayer it
+    only lends its factor, to the kernel that adds the result to the stream.
+
+    params: `size`.  tensors: `weight` [size]."""
+
+    def local_weights(self):
+        return {"weight": ((int(self.params["size"]),), "norm")}
+
+    def prepare(self, dtype, device) -> None:
+        self.factor = self.tensors["weight"].to(torch.float32).contiguous()
