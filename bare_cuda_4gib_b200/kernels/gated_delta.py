@@ -103,3 +103,55 @@ def step(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, gates: 
         {"silu": 1, "sigmoid": 0}[gate_kind], norm_w.data_ptr(), out.data_ptr(), out.stride(0), ctx.positions.data_ptr(),
         ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.n_seqs, heads, kv_heads, dk, dv, 1 if write_ring else 0,
         float(unit_eps), dk ** -0.5, float(eps), ctx.stream), "gated_delta_step")
+
+
+CHUNKED_MIN_TOKENS = 32      # steps with a portion at least this long take the chunked walk
+CHUNK = 64
+_chunked_libs = {}
+
+
+def chunked_takes(dk: int, dv: int) -> bool:
+    """Head sizes the chunked walk on the tensor cores takes (a library per key size)."""
+    return dk % 16 == 0 and 16 <= dk <= 128 and dv % 16 == 0
+
+
+def chunked_columns(heads: int, dv: int) -> int:
+    """Value columns of a block: 32, or 16 where one request's blocks would not come near the number of SMs."""
+    from .lib import sm_count
+    return 32 if dv % 32 == 0 and heads * (dv // 32) >= sm_count() // 2 else 16
+
+
+def chunked_lib(dk: int):
+    l = _chunked_libs.get(dk)
+    if l is None:
+        l = build.load_library("gated_delta_chunked.cu", (f"-DGD_DK={dk}",))
+        P, I, L = c_void_p, c_int, c_longlong
+        l.llm_gated_delta_prepare.argtypes = [P, P, P, P, L, I, P, L, I, P, P, I, P, P, P, L, P, L, P, P, P, P, I, I, I, I, I, I, P]
+        l.llm_gated_delta_walk.argtypes = [P, P, P, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]
+        l.llm_gated_delta_prepare.restype = l.llm_gated_delta_walk.restype = c_int
+        _chunked_libs[dk] = l
+    return l
+
+
+def chunked(ctx, qn: torch.Tensor, kn: torch.Tensor, vn: torch.Tensor, gates: Gates, state: torch.Tensor, out: torch.Tensor,
+            heads: int, kv_heads: int, dk: int, dv: int, columns: int = 0) -> None:
+    """What `scan` does, in chunks of 64 tokens on the tensor cores: two kernels, one over all chunks side by side
+    for everything that does not depend on the state, one that walks every request's chunks in order."""
+    _floats("chunked", qn, kn, vn, state, out)
+    columns = columns or chunked_columns(heads, dv)
+    n = ctx.n_tokens
+    tiles = ctx.ws.get("delta_tiles", (6, n, heads * dk), torch.bfloat16, max_lead=6)      # (W, Q', K'') x (rounded, rest)
+    pairs = ctx.ws.get("delta_pairs", (2, n, heads * CHUNK), torch.bfloat16, max_lead=2)
+    u = ctx.ws.get("delta_u", (n, heads * dv), torch.float32)
+    most = ctx.max_rows // CHUNK + ctx.max_seqs + 1
+    end = ctx.ws.get("delta_end", (n // CHUNK + ctx.n_seqs + 1, heads * dk), torch.float32, max_rows=most)
+    l = chunked_lib(dk)
+    plane = tiles.stride(0)
+    at = [tiles.data_ptr() + 2 * plane * i for i in range(6)]
+    where = (at[0], at[1], at[2], 3 * plane, pairs.data_ptr(), pairs.stride(0), u.data_ptr(), end.data_ptr())
+    _check(l.llm_gated_delta_prepare(
+        qn.data_ptr(), kn.data_ptr(), vn.data_ptr(), *gates.arguments(), *where, ctx.seq_q_start.data_ptr(),
+        ctx.seq_q_len.data_ptr(), ctx.n_seqs, int(ctx.max_q_len), heads, kv_heads, dk, dv, ctx.stream), "gated_delta_prepare")
+    _check(l.llm_gated_delta_walk(
+        *where, state.data_ptr(), out.data_ptr(), ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(),
+        ctx.seq_q_len.data_ptr(), ctx.n_seqs, heads, dk, dv, columns, ctx.stream), "gated_delta_walk")

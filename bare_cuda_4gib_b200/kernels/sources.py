@@ -12,7 +12,8 @@ def all_libraries():
             ("latent_attention.cu", ()), ("mlstm.cu", ()), ("diff_attention.cu", ()), ("moe.cu", ()),
             ("gated_sandwich.cu", ()), ("mamba2.cu", ()),
             ("mamba2_chunked.cu", ("-DSSD_N=128", "-DSSD_P=64", "-DSSD_PC=16")),
-            ("mamba2_chunked.cu", ("-DSSD_N=128", "-DSSD_P=64", "-DSSD_PC=32"))]
+            ("mamba2_chunked.cu", ("-DSSD_N=128", "-DSSD_P=64", "-DSSD_PC=32")),
+            ("gated_delta.cu", ()), ("gated_delta_chunked.cu", ("-DGD_DK=16",)), ("gated_delta_chunked.cu", ("-DGD_DK=128",))]
     jobs += [("gemm_tcgen05.cu", ("-DGLU_GELU_TANH",)), ("gemv_fused.cu", ("-DGLU_GELU_TANH",)),
              ("gemm_tcgen05.cu", ("-DGROUPED_UP_RELU2",))]
     jobs += [("attention_mma.cu", (f"-DHEAD_DIM={d}",)) for d in ATTENTION_HEAD_DIMS]

@@ -153,6 +153,28 @@ PRESETS.update({
 })
 
 
+def _sizitar(width, vocab, ff, heads, kv_heads, dim, conv, state_heads, state_kv, state_dim, rank, experts, top, expert_ff,
+             loop):
+    """A delta layer with a dense feed-forward, then channel_delta, attention and channel_delta layers with experts."""
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": expert_ff}}
+    state = {"dim": state_dim, "vdim": state_dim, "conv": conv}
+    delta = {"type": "delta", "mlp": {"kind": "dense", "ff": ff}, "mixer": dict(state, heads=state_heads, kv_heads=state_kv)}
+    channel = {"type": "channel_delta", "mlp": mlp, "mixer": dict(state, heads=state_heads, kv_heads=state_heads, rank=rank)}
+    attention = {"type": "attention", "mlp": mlp,
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv, "scale": dim ** -0.5,
+                           "rot": {"base": 10000.0, "dims": dim // 2}}}
+    return dict(architecture="Sizitar", vocab=vocab, width=width, norm={"eps": 1e-6}, logit_scale=0.5, loop=loop,
+                layers=[delta, channel, attention, channel])
+
+
+PRESETS.update({
+    "sizitar-tiny": _sizitar(64, 300, 96, 4, 2, 16, 3, 4, 2, 16, 8, 5, 2, 32, {"start": 1, "stop": 3, "times": 2}),
+    # widths and expert sizes of the Gurolix presets; heads of 128 everywhere, states as large as theirs
+    "sizitar-2048": _sizitar(2048, 32000, 5632, 16, 4, 128, 4, 32, 16, 128, 128, 8, 2, 1408, None),
+    "sizitar-4096": _sizitar(4096, 32000, 11008, 32, 8, 128, 4, 64, 32, 128, 128, 8, 2, 2752, None),
+})
+
+
 def preset_config(name: str, **overrides):
     from ..config.llama import LlamaConfig
     from ..errors import ConfigError

@@ -117,6 +117,9 @@ class GatedDelta(Part):
             if first % 8 == 0 and width % 8 == 0:
                 self.expand.prepare(dtype)
         self.one_step = device.type == "cuda" and GD.step_takes(self.dim, self.vdim)
+        self.chunked = device.type == "cuda" and dtype == torch.bfloat16 and GD.chunked_takes(self.dim, self.vdim)
+        if self.chunked:
+            GD.chunked_lib(self.dim)      # compiled with the model, not at its first long portion
         self.tensors = {}
 
     def forward(self, ctx, call, h):
@@ -144,6 +147,9 @@ class GatedDelta(Part):
         if call.writes_cache:
             from ..kernels import mamba2 as MK
             MK.ring_write(ctx, u[:, : self.conv_channels], ring, self.taps, self.conv_channels)
-        GD.scan(ctx, qn, kn, vn, gates, state, scanned, H, G, dk, dv)
+        if self.chunked and ctx.max_q_len >= GD.CHUNKED_MIN_TOKENS and ctx.use_fast_attention:
+            GD.chunked(ctx, qn, kn, vn, gates, state, scanned, H, G, dk, dv)
+        else:
+            GD.scan(ctx, qn, kn, vn, gates, state, scanned, H, G, dk, dv)
         LA.gated_group_norm(scanned, gate, self.norm_w, out, n, dv, self.gate_kind, self.eps, 1.0, ctx.stream)
         return self.o.forward(ctx, out, n, f32, "mixer_out", allow_partials=True)

@@ -186,9 +186,10 @@ SETTLE_SECONDS = 0.1      # pause between putting the prompts into the cache and
 
 
 def design_main(args) -> int:
-    """`--design dopudra`, `zadurax`, `pudulorn`, `gurolix` or `fuzazen`: one JSON line with, per size, a prefill step of `--prefill-tokens` tokens and decode
+    """`--design dopudra`, `zadurax`, `pudulorn`, `gurolix`, `fuzazen` or `sizitar`: one JSON line with, per size, a prefill step of `--prefill-tokens` tokens and decode
     steps at `--batch` requests of `--context` positions for the design and for the Llama decoder of the same
-    width (for `gurolix`: the Pudulorn decoder, the engine's other design with a mixture of experts; for
+    width (for `gurolix`: the Pudulorn decoder, the engine's other design with a mixture of experts; for `sizitar`: the
+    Gurolix decoder, the other one with matrix states and ungated experts; for
     `fuzazen` a third size with value heads of their own size beside the Llama decoder of that width), both with
     `--design-layers` layers, seeded random weights, bfloat16, CUDA events around the steps."""
     import torch
@@ -259,7 +260,7 @@ def design_main(args) -> int:
                 "weight_bytes": weights}
 
     sizes = []
-    beside = {"gurolix": ("pudulorn-2048", "pudulorn-4096")}.get(args.design, ("tinyllama", "llama2-7b"))
+    beside = {"gurolix": ("pudulorn-2048", "pudulorn-4096"), "sizitar": ("gurolix-2048", "gurolix-4096")}.get(args.design, ("tinyllama", "llama2-7b"))
     pairs = [(f"{args.design}-2048", beside[0]), (f"{args.design}-4096", beside[1])]
     if args.design == "fuzazen":
         pairs.append(("fuzazen-2048-values", beside[0]))
@@ -297,7 +298,7 @@ def main() -> int:
     ap.add_argument("--no-graphs", action="store_true")
     ap.add_argument("--only", default="", choices=["", "prefill", "decode"],
                     help="profiling aid: run just the prefill step or just the decode steps and print their time")
-    ap.add_argument("--design", default="", choices=["", "dopudra", "zadurax", "pudulorn", "gurolix", "fuzazen"],
+    ap.add_argument("--design", default="", choices=["", "dopudra", "zadurax", "pudulorn", "gurolix", "fuzazen", "sizitar"],
                     help="instead of the default workload: prefill and decode throughput of this design at layer sizes "
                          "of real models, beside the Llama decoder at equal width, layer count and vocabulary")
     ap.add_argument("--design-layers", type=int, default=8, help="layers of both models in a --design run")
