@@ -13,6 +13,7 @@
 // softmax and the weighted sum are float32.
 
 #include "common.cuh"
+#include "short_conv.cuh"
 
 #include <math.h>
 
@@ -121,14 +122,103 @@ __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restric
   }
 }
 
+// The same for bfloat16 in pieces of four channels: sizes that are multiples of four, up to four taps, a rotation in
+// neighbouring pairs or none.  A block walks `rows_per_block` rows with its channels' weights and last inputs in
+// registers, PIECES pieces a thread.  With `write_ring` (steps of one token per request only) it also does what
+// conv_ring_write does: the entry it writes is the one the same thread has read as the oldest input.
+template <int TAPS, int PIECES>
+__global__ void __launch_bounds__(PIECES == 1 ? 1024 : 768)
+conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, const float* __restrict__ conv_w,
+                           float* __restrict__ ring, const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w,
+                           __nv_bfloat16* __restrict__ q_out, PagedCacheKV cache, const int32_t* __restrict__ positions,
+                           const int32_t* __restrict__ row_seq, const int32_t* __restrict__ seq_slot,
+                           const int32_t* __restrict__ seq_q_start, int n_tokens, int rows_per_block, int qd, int kd, int vd,
+                           float eps, float temp_coef, int temp_every, int write_cache, int write_ring,
+                           const float* __restrict__ inv_freq, int rot_dims) {
+  pdl_launch_dependents();
+  extern __shared__ float turns[];             // [2][rot_dims] cosines, then sines, of two rows in turn
+  __shared__ float2 sums[2][32];
+  constexpr int HIST = TAPS - 1;
+  const int C = qd + kd + vd, half = rot_dims / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n_warps = blockDim.x >> 5;
+  ConvColumns<TAPS> conv[PIECES];
+  int at[PIECES];
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    at[j] = (threadIdx.x + j * blockDim.x) * 4;
+    if (at[j] < C) conv[j].load_weights(conv_w, at[j]);
+  }
+  pdl_wait();
+  const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, n_tokens - t0);
+  int seq = -1;
+  for (int r = 0; r < rows; ++r) {
+    const int t = t0 + r, s = row_seq[t], p = positions[t], parity = r & 1;
+    float* turn = turns + parity * rot_dims;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)p * inv_freq[i], &turn[half + i], &turn[i]);
+    const bool fresh = s != seq;
+    seq = s;
+    float* ring_slot = ring + (long long)seq_slot[s] * (HIST > 0 ? HIST : 1) * C;
+    float y[PIECES][4];
+    float2 sq = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j) {
+      if (at[j] >= C) continue;
+      if (fresh) conv[j].history(u, u_stride, at[j], t, p, seq_q_start[s], ring_slot, HIST, C);
+      const uint2 now = conv_load4(u + (long long)t * u_stride + at[j]);
+      conv[j].step(now, y[j]);
+      if (HIST > 0 && write_ring) *reinterpret_cast<float4*>(ring_slot + (long long)(p % (HIST > 0 ? HIST : 1)) * C + at[j]) = conv_floats(now);
+      const float e = y[j][0] * y[j][0] + y[j][1] * y[j][1] + y[j][2] * y[j][2] + y[j][3] * y[j][3];
+      if (at[j] < qd) sq.x += e;
+      else if (at[j] < qd + kd) sq.y += e;
+    }
+    sq.x = warp_sum(sq.x);
+    sq.y = warp_sum(sq.y);
+    if (lane == 0) sums[parity][warp] = sq;
+    __syncthreads();      // (two rows' sums and turns in turn: a row's are written again behind the next row's barrier)
+    sq = lane < n_warps ? sums[parity][lane] : make_float2(0.0f, 0.0f);
+    const float rq = 1.0f / sqrtf(warp_sum(sq.x) / (float)qd + eps) * (1.0f + temp_coef * logf((float)((p + 1) / temp_every + 1)));
+    const float rk = 1.0f / sqrtf(warp_sum(sq.y) / (float)kd + eps);
+    const int page = cache_page(cache, s, p), in_page = p % cache.page_tokens;
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j) {
+      if (at[j] >= C) continue;
+      __nv_bfloat16* dst;
+      if (at[j] < qd + kd) {
+        const bool is_q = at[j] < qd;
+        const int e = is_q ? at[j] : at[j] - qd, head = e / cache.k_dim, d = e - head * cache.k_dim;
+        const float4 w = *reinterpret_cast<const float4*>((is_q ? q_norm_w : k_norm_w) + e);
+        const float f = is_q ? rq : rk;
+        y[j][0] *= f * w.x; y[j][1] *= f * w.y; y[j][2] *= f * w.z; y[j][3] *= f * w.w;
+#pragma unroll
+        for (int x = 0; x < 4; x += 2) {
+          if (d + x < rot_dims) {
+            const float c = turn[(d + x) / 2], sn = turn[half + (d + x) / 2], a = y[j][x], b = y[j][x + 1];
+            y[j][x] = a * c - b * sn;
+            y[j][x + 1] = b * c + a * sn;
+          }
+        }
+        dst = is_q ? q_out + (long long)t * qd + e
+                   : (__nv_bfloat16*)cache.k + (long long)page * cache.page_stride + ((long long)head * cache.page_tokens + in_page) * cache.k_dim + d;
+        if (!is_q && (!write_cache || page < 0)) continue;
+      } else {
+        const int e = at[j] - qd - kd, head = e / cache.v_dim, d = e - head * cache.v_dim;
+        if (!write_cache || page < 0) continue;
+        dst = (__nv_bfloat16*)cache.v + (long long)page * cache.page_stride + ((long long)head * cache.page_tokens + in_page) * cache.v_dim + d;
+      }
+      *reinterpret_cast<uint2*>(dst) = conv_pack4(y[j]);
+    }
+  }
+}
+
 extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride, const float* conv_w, int taps,
-                                   const float* ring, const float* q_norm_w, const float* k_norm_w, void* q_out,
+                                   float* ring, const float* q_norm_w, const float* k_norm_w, void* q_out,
                                    void* cache_k, void* cache_v, const int32_t* block_table, long long page_stride,
                                    int table_stride, int page_tokens, int kv_heads, int k_dim, int v_dim,
                                    const int32_t* positions, const int32_t* row_seq, const int32_t* seq_slot,
                                    const int32_t* seq_q_start, int n_tokens, int q_heads, float eps, float temp_coef,
                                    int temp_every, int write_cache, const float* inv_freq, int rot_dims, int halves,
-                                   cudaStream_t stream) {
+                                   int write_ring, int* ring_written, cudaStream_t stream) {
+  *ring_written = 0;
   if (n_tokens <= 0) return 0;
   LLM_HOST_CHECK(taps >= 1 && temp_every >= 1, ERR_BAD_SIZE);
   if (!inv_freq) rot_dims = 0;
@@ -139,6 +229,29 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
   LLM_HOST_CHECK(smem <= 200 * 1024, ERR_BAD_SIZE);
   const int threads = C >= 2048 ? 512 : (C >= 512 ? 256 : 128);
   PagedCacheKV cache{cache_k, cache_v, block_table, page_stride, table_stride, page_tokens, kv_heads, k_dim, v_dim};
+  auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
+  const int pieces = C / 4 <= 1024 ? 1 : 2;
+  const bool vec = dtype == DT_BF16 && taps <= 4 && !(halves && rot_dims) && k_dim % 4 == 0 && v_dim % 4 == 0 &&
+                   C / 4 <= 2 * 768 && u_stride % 4 == 0 && page_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) &&
+                   aligned(q_norm_w, 16) && aligned(k_norm_w, 16) && aligned(q_out, 8) && aligned(cache_k, 8) && aligned(cache_v, 8);
+  if (vec) {
+    *ring_written = write_ring;
+    const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 1024 ? 8 : (n_tokens >= 256 ? 2 : 1);
+    const int blocks = (n_tokens + per_block - 1) / per_block;
+#define VEC(TAPS, PIECES)                                                                                              \
+  launch_kernel(conv_norm_cache_vec_kernel<TAPS, PIECES>, blocks, wide, (size_t)2 * rot_dims * sizeof(float), stream,  \
+                (const __nv_bfloat16*)u, u_stride, conv_w, ring, q_norm_w, k_norm_w, (__nv_bfloat16*)q_out, cache,      \
+                positions, row_seq, seq_slot, seq_q_start, n_tokens, per_block, qd, kd, vd, eps, temp_coef, temp_every, \
+                write_cache, write_ring, inv_freq, rot_dims)
+#define TAPS_OF(PIECES)                                                                                                \
+  do {                                                                                                                 \
+    if (taps == 1) VEC(1, PIECES); else if (taps == 2) VEC(2, PIECES); else if (taps == 3) VEC(3, PIECES); else VEC(4, PIECES); \
+  } while (0)
+    if (pieces == 1) TAPS_OF(1); else TAPS_OF(2);
+#undef TAPS_OF
+#undef VEC
+    return launch_status();
+  }
 #define LAUNCH(T)                                                                                                 \
   do {                                                                                                            \
     if (smem > 48 * 1024)                                                                                         \
@@ -155,32 +268,32 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
 }
 
 // The projection rows of each request's last taps - 1 positions go into its ring (entry position %
-// (taps - 1)), after the convolution of the step has read the ring.
+// (taps - 1)), after the convolution of the step has read the ring.  Grid (request x kept position, slice of channels).
 template <typename T>
 __global__ void conv_ring_write_kernel(const T* __restrict__ u, long long u_stride, float* __restrict__ ring, int hist,
-                                       int C, const int32_t* __restrict__ positions, const int32_t* __restrict__ row_seq,
-                                       const int32_t* __restrict__ seq_slot, const int32_t* __restrict__ seq_kv_len) {
+                                       int C, const int32_t* __restrict__ seq_slot, const int32_t* __restrict__ seq_q_start,
+                                       const int32_t* __restrict__ seq_q_len, const int32_t* __restrict__ seq_kv_len) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x;
-  const int seq = row_seq[t], p = positions[t];
-  const int end = seq_kv_len[seq] > 0 ? seq_kv_len[seq] : p + 1;   // an idle row stands for itself
-  if (p < end - hist) return;
+  const int seq = blockIdx.x / hist, back = blockIdx.x % hist + 1;      // the request's last position, the last but one, ...
+  if (back > seq_q_len[seq]) return;
+  const int t = seq_q_start[seq] + seq_q_len[seq] - back, p = seq_kv_len[seq] - back;
   float* dst = ring + ((long long)seq_slot[seq] * hist + (p % hist)) * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = to_float(u[(long long)t * u_stride + c]);
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
+    dst[c] = to_float(u[(long long)t * u_stride + c]);
 }
 
 extern "C" int llm_conv_ring_write(const void* u, int dtype, long long u_stride, float* ring, int taps, int channels,
-                                   const int32_t* positions, const int32_t* row_seq, const int32_t* seq_slot,
-                                   const int32_t* seq_kv_len, int n_tokens, cudaStream_t stream) {
-  if (n_tokens <= 0 || taps <= 1) return 0;
-  const int threads = channels >= 1024 ? 256 : 128;
+                                   const int32_t* seq_slot, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                                   const int32_t* seq_kv_len, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0 || taps <= 1) return 0;
+  const dim3 grid(n_seqs * (taps - 1), (channels + 1023) / 1024);
   if (dtype == DT_F32)
-    launch_kernel(conv_ring_write_kernel<float>, n_tokens, threads, 0, stream, (const float*)u, u_stride, ring,
-                  taps - 1, channels, positions, row_seq, seq_slot, seq_kv_len);
+    launch_kernel(conv_ring_write_kernel<float>, grid, 256, 0, stream, (const float*)u, u_stride, ring, taps - 1, channels,
+                  seq_slot, seq_q_start, seq_q_len, seq_kv_len);
   else if (dtype == DT_BF16)
-    launch_kernel(conv_ring_write_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, (const __nv_bfloat16*)u,
-                  u_stride, ring, taps - 1, channels, positions, row_seq, seq_slot, seq_kv_len);
+    launch_kernel(conv_ring_write_kernel<__nv_bfloat16>, grid, 256, 0, stream, (const __nv_bfloat16*)u, u_stride, ring,
+                  taps - 1, channels, seq_slot, seq_q_start, seq_q_len, seq_kv_len);
   else
     return ERR_BAD_DTYPE;
   return launch_status();

@@ -7,7 +7,8 @@
 // short causal convolution per channel and silu; q and k are then divided by sqrt(sum of squares + unit_eps) per
 // head, q also by sqrt(dk).  `heads` value heads share `kv_heads` query/key heads (head h reads h / (heads / kv_heads)).
 //
-// Kernels: gated_delta_operands (convolution, silu, unit vectors: float32 q, k, v of a step's tokens),
+// Kernels: gated_delta_operands (convolution, silu, unit vectors: float32 q, k, v of a step's tokens, or for the
+// chunked walk the activations in bfloat16 with the unit vectors' factors beside them),
 // gated_delta_scan (the walk over a step's tokens, any sizes, float32), gated_delta_step (steps of one token
 // per request: convolution with the ring's update, unit vectors, decays, the state in place, the norm per head
 // and the output gate in one kernel).  Long portions of bfloat16 steps take gated_delta_chunked.cu instead of
@@ -15,17 +16,21 @@
 // by position % taps.  Everything after the stored projections is float32.
 
 #include "gated_delta.cuh"
+#include "short_conv.cuh"
 
 // ------------------------------------------------------------------------------------------- operands
 
-// One block per token.  u: the projection's rows [q: G dk | k: G dk | v: H dv | ...].
+// One block per token.  u: the projection's rows [q: G dk | k: G dk | v: H dv | ...].  With `compact`: the
+// activations rounded to bfloat16, [rows][q | k | v], and in `lengths` [rows][2 G] what makes unit vectors of the
+// rounded q and k heads, 1 / sqrt(sum of squares + unit_eps), of q also / sqrt(dk).
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_delta_operands_kernel(const T* __restrict__ u, long long u_stride, const float* __restrict__ conv_w, int taps,
                             const float* __restrict__ ring, float* __restrict__ qn, float* __restrict__ kn,
                             float* __restrict__ vn, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ row_seq, const int32_t* __restrict__ seq_slot,
-                            const int32_t* __restrict__ seq_q_start, int G, int dk, int vd, float unit_eps, float q_scale) {
+                            const int32_t* __restrict__ seq_q_start, int G, int dk, int vd, float unit_eps, float q_scale,
+                            __nv_bfloat16* __restrict__ compact, float* __restrict__ lengths) {
   pdl_launch_dependents();
   extern __shared__ float ys[];      // [2 G dk] q and k after convolution and silu
   const int kd = G * dk, C = 2 * kd + vd;
@@ -51,7 +56,13 @@ gated_delta_operands_kernel(const T* __restrict__ u, long long u_stride, const f
       }
     }
     y = delta_silu(y);
+    if (compact) {
+      const __nv_bfloat16 r = __float2bfloat16_rn(y);
+      compact[(long long)t * C + c] = r;
+      y = __bfloat162float(r);
+    }
     if (c < 2 * kd) ys[c] = y;
+    else if (compact) continue;
     else vn[(long long)t * vd + (c - 2 * kd)] = y;
   }
   __syncthreads();
@@ -61,8 +72,59 @@ gated_delta_operands_kernel(const T* __restrict__ u, long long u_stride, const f
     float sq = 0.0f;
     for (int i = lane; i < dk; i += 32) sq += x[i] * x[i];
     const float s = (head < G ? q_scale : 1.0f) / sqrtf(warp_sum(sq) + unit_eps);
+    if (compact) {
+      if (lane == 0) lengths[(long long)t * 2 * G + head] = s;
+      continue;
+    }
     float* dst = (head < G ? qn + (long long)t * kd + head * dk : kn + (long long)t * kd + (head - G) * dk);
     for (int i = lane; i < dk; i += 32) dst[i] = x[i] * s;
+  }
+}
+
+// The compact form with a thread per four channels that walks OPER_ROWS rows: bfloat16, key heads of 16 to 128
+// entries (a power of two, so that a head's lanes sum its squares by shuffles), value sizes that are multiples of four.
+#define OPER_ROWS 16
+#define OPER_THREADS 128
+
+template <int TAPS>
+__global__ void __launch_bounds__(OPER_THREADS)
+gated_delta_compact_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, const float* __restrict__ conv_w,
+                           const float* __restrict__ ring, const int32_t* __restrict__ positions,
+                           const int32_t* __restrict__ row_seq, const int32_t* __restrict__ seq_slot,
+                           const int32_t* __restrict__ seq_q_start, int n_tokens, int G, int dk, int vd, float unit_eps,
+                           float q_scale, __nv_bfloat16* __restrict__ compact, float* __restrict__ lengths) {
+  pdl_launch_dependents();
+  const int kd = G * dk, C = 2 * kd + vd;
+  const int c = (blockIdx.y * OPER_THREADS + threadIdx.x) * 4;
+  const bool live = c < C;
+  const int cc = live ? c : 0;      // (idle lanes follow along on the first channels: the shuffles need every lane)
+  ConvColumns<TAPS> conv;
+  conv.load_weights(conv_w, cc);
+  pdl_wait();
+  const int t0 = blockIdx.x * OPER_ROWS, rows = min(OPER_ROWS, n_tokens - t0);
+  const int lanes = dk / 4;
+  int seq = -1;
+  for (int i0 = 0; i0 < rows; i0 += 4) {      // four rows' inputs are asked for together
+    uint2 in[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) in[k] = conv_load4(u + (long long)(t0 + min(i0 + k, rows - 1)) * u_stride + cc);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (i0 + k >= rows) break;
+      const int t = t0 + i0 + k, s = row_seq[t];
+      if (s != seq) {
+        seq = s;
+        conv.history(u, u_stride, cc, t, positions[t], seq_q_start[s], ring + (long long)seq_slot[s] * TAPS * C, TAPS, C);
+      }
+      float y[4];
+      conv.step(in[k], y);
+#pragma unroll
+      for (int x = 0; x < 4; ++x) y[x] = __bfloat162float(__float2bfloat16_rn(delta_silu(y[x])));
+      if (live) *reinterpret_cast<uint2*>(compact + (long long)t * C + c) = conv_pack4(y);
+      float sq = y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3];
+      for (int o = lanes >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      if (live && c < 2 * kd && c % dk == 0) lengths[(long long)t * 2 * G + c / dk] = (c < kd ? q_scale : 1.0f) / sqrtf(sq + unit_eps);
+    }
   }
 }
 
@@ -70,17 +132,32 @@ extern "C" int llm_gated_delta_operands(const void* u, int dtype, long long u_st
                                         const float* ring, float* qn, float* kn, float* vn, const int32_t* positions,
                                         const int32_t* row_seq, const int32_t* seq_slot, const int32_t* seq_q_start,
                                         int n_tokens, int kv_heads, int dk, int heads, int dv, float unit_eps, float q_scale,
-                                        cudaStream_t stream) {
+                                        void* compact, float* lengths, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  LLM_HOST_CHECK(!compact || lengths, ERR_BAD_SIZE);
   LLM_HOST_CHECK(taps >= 1 && kv_heads >= 1 && dk >= 1 && heads >= 1 && dv >= 1, ERR_BAD_SIZE);
   const size_t smem = (size_t)2 * kv_heads * dk * sizeof(float);
   LLM_HOST_CHECK(smem <= 200 * 1024, ERR_BAD_SIZE);
+  auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
+  if (compact && dtype == DT_BF16 && taps <= 4 && dk >= 16 && dk <= 128 && (dk & (dk - 1)) == 0 && dv % 4 == 0 &&
+      u_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) && aligned(compact, 8)) {
+    const int C = 2 * kv_heads * dk + heads * dv;
+    const dim3 grid((n_tokens + OPER_ROWS - 1) / OPER_ROWS, (C / 4 + OPER_THREADS - 1) / OPER_THREADS);
+#define COMPACT(TAPS)                                                                                                 \
+  launch_kernel(gated_delta_compact_kernel<TAPS>, grid, OPER_THREADS, 0, stream, (const __nv_bfloat16*)u, u_stride,    \
+                conv_w, ring, positions, row_seq, seq_slot, seq_q_start, n_tokens, kv_heads, dk, heads * dv, unit_eps, \
+                q_scale, (__nv_bfloat16*)compact, lengths)
+    if (taps == 1) COMPACT(1); else if (taps == 2) COMPACT(2); else if (taps == 3) COMPACT(3); else COMPACT(4);
+#undef COMPACT
+    return launch_status();
+  }
 #define LAUNCH(T)                                                                                                       \
   do {                                                                                                                  \
     if (smem > 48 * 1024)                                                                                               \
       cudaFuncSetAttribute(gated_delta_operands_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     launch_kernel(gated_delta_operands_kernel<T>, n_tokens, 256, smem, stream, (const T*)u, u_stride, conv_w, taps, ring, \
-                  qn, kn, vn, positions, row_seq, seq_slot, seq_q_start, kv_heads, dk, heads * dv, unit_eps, q_scale);   \
+                  qn, kn, vn, positions, row_seq, seq_slot, seq_q_start, kv_heads, dk, heads * dv, unit_eps, q_scale,    \
+                  (__nv_bfloat16*)compact, lengths);                                                                    \
   } while (0)
   if (dtype == DT_F32) LAUNCH(float);
   else if (dtype == DT_BF16) LAUNCH(__nv_bfloat16);

@@ -15,9 +15,10 @@
 // another.  Decays are differences of logarithms that are never positive, so no factor overflows: a block of 16 x
 // 16 pairs of tokens takes its factors against the last token ahead of its rows, exp(c_t - r) exp(r - c_j); inside a
 // block on the diagonal the second one can grow, and where it would leave float32's range the pairs are formed
-// one by one.  Every product's operands are two bfloat16 numbers each, a rounded one and what rounding left, of
-// whose four products the three large ones are taken: 16 significant bits.  L's inverse, the decays and the state
-// are float32.
+// one by one.  (One decay for all channels is a factor of the pair, behind an exact product of bfloat16 rows.)
+// q, k and v arrive as bfloat16 activations, q and k with the float32 factors that make unit vectors of them.
+// Every other operand of a product is two bfloat16 numbers, a rounded one and what rounding left, of whose four
+// products the three large ones are taken: 16 significant bits.  Sums, decays and the state are float32.
 //
 // Built per key size with -DGD_DK (a multiple of 16 up to 128).
 
@@ -32,10 +33,6 @@ namespace {
 constexpr int DK = GD_DK;
 static_assert(DK % 16 == 0 && DK >= 16 && DK <= 128, "GD_DK must be a multiple of 16 up to 128");
 constexpr int L = 64;                  // tokens of a chunk
-constexpr int LDF = DK + 4;            // float rows in shared memory
-constexpr int LDT = L + 4;
-constexpr int PREP_THREADS = 512;
-constexpr float SAFE_RANGE = 80.0f;    // exp(80) times a chunk's sums stays inside float32
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
 
@@ -85,24 +82,52 @@ __device__ __forceinline__ long long chunk_id(int q_start, int seq, int chunk) {
 
 // ------------------------------------------------------------------------------------------- prepare
 
-template <bool CHANNEL>
-struct PrepShared {
-  static constexpr int C_FLOATS = CHANNEL ? L * LDF : L;
-  static constexpr size_t BYTES = sizeof(float) * (size_t)(2 * L * LDF + C_FLOATS + L * LDT + L);
-};
+constexpr int PREP_THREADS = 256;
+constexpr int LDN = DK + 8;            // padded bfloat16 rows (conflict-free ldmatrix)
+constexpr int LDF = DK + 4;            // float rows
+constexpr int LDL = L + 4;             // float rows of L
+constexpr int LDP = L + 8;             // bfloat16 rows of T and P
+constexpr int LDD = 24;                // bfloat16 rows of a block on T's diagonal
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr float SAFE_RANGE = 100.0f;   // 2^100 times a sum over the key channels stays inside float32
 
 template <bool CHANNEL>
-__global__ void __launch_bounds__(PREP_THREADS)
-gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vn,
-                           DeltaGates gates, Tiles o, const int32_t* __restrict__ seq_q_start,
-                           const int32_t* __restrict__ seq_q_len, int H, int G, int dv) {
+struct PrepShared {      // in bytes
+  static constexpr size_t TILE = (size_t)L * LDN * 2;                    // k or q; later one part of K'
+  static constexpr size_t SUMS = CHANNEL ? (size_t)L * LDF * 4 : L * 4 + TILE;      // sums of logarithms; later (or behind them) values
+  static constexpr size_t BYTES = 2 * TILE + SUMS + (size_t)L * LDL * 4 + 2 * (size_t)L * LDP * 2 + 2 * 4 * 16 * LDD * 2 + 3 * L * 4;
+};
+
+// Blocks of three products of two-part operands.
+__device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0,
+                                          uint32_t bh1, uint32_t bl0, uint32_t bl1) {
+  mma_bf16(c, ah, bh0, bh1);
+  mma_bf16(c, al, bh0, bh1);
+  mma_bf16(c, ah, bl0, bl1);
+}
+
+__device__ __forceinline__ float2 pair_of(const __nv_bfloat16* p) {
+  const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(p);
+  return make_float2(__low2float(v), __high2float(v));
+}
+
+template <bool CHANNEL>
+__global__ void __launch_bounds__(PREP_THREADS, 2)
+gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* __restrict__ lengths, DeltaGates gates, Tiles o,
+                           const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_q_len, int H, int G, int dv) {
   pdl_launch_dependents();
-  extern __shared__ __align__(16) float sm[];
-  float* ks = sm;                                        // [L][LDF] k, later K'
-  float* qs = ks + L * LDF;                              // [L][LDF]
-  float* cs = qs + L * LDF;                              // [L][LDF] sums of logarithms, or [L]
-  float* Lm = cs + PrepShared<CHANNEL>::C_FLOATS;        // [L][LDT] L, later (1 + L)^-1
-  float* betas = Lm + L * LDT;                           // [L]
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  using Sh = PrepShared<CHANNEL>;
+  __nv_bfloat16* kt = reinterpret_cast<__nv_bfloat16*>(smem_raw);                  // [L][LDN] k; later K' rounded
+  __nv_bfloat16* qt = kt + L * LDN;                                                // [L][LDN] q; later what rounding K' left
+  float* cs = reinterpret_cast<float*>(smem_raw + 2 * Sh::TILE);                   // [L][LDF] or [L], in units of log 2
+  __nv_bfloat16* vt = reinterpret_cast<__nv_bfloat16*>(cs + (CHANNEL ? 0 : L));    // [L][LDN] a piece of the values
+  float* Lm = reinterpret_cast<float*>(smem_raw + 2 * Sh::TILE + Sh::SUMS);        // [L][LDL]
+  __nv_bfloat16* T = reinterpret_cast<__nv_bfloat16*>(Lm + L * LDL);               // [2][L][LDP] T: rounded, rest
+  __nv_bfloat16* D = T + 2 * L * LDP;                                              // [2][4][16][LDD] (1 + L)^-1's diagonal blocks
+  float* betas = reinterpret_cast<float*>(D + 2 * 4 * 16 * LDD);                   // [L]
+  float* k_len = betas + L;                                                        // [L] factors that make unit vectors
+  float* q_len_ = k_len + L;                                                       // [L]
   pdl_wait();
   const int chunk = blockIdx.x, h = blockIdx.y, seq = blockIdx.z;
   const int q_len = seq_q_len[seq];
@@ -110,16 +135,18 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
   const int count = min(L, q_len - chunk * L), q_start = seq_q_start[seq];
   const long long row0 = q_start + (long long)chunk * L;
   const int g = h / (H / G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int gq = lane >> 2, tq = lane & 3;
-  const float neg_a = -expf(gates.a_log[h]);
+  const int gq = lane >> 2, tq = lane & 3, mid = lane >> 3;
+  const long long C = 2LL * G * DK + (long long)H * dv;      // columns of qkv
+  const float neg_a = -LOG2E * expf(gates.a_log[h]);
 
-  for (int e = tid; e < L * (DK / 4); e += PREP_THREADS) {
-    const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+  for (int e = tid; e < L * (DK / 8); e += PREP_THREADS) {
+    const int t = e / (DK / 8), c = (e % (DK / 8)) * 8;
     const bool in = t < count;
-    const long long src = (row0 + t) * ((long long)G * DK) + g * DK + c;
-    *reinterpret_cast<float4*>(ks + t * LDF + c) = in ? *reinterpret_cast<const float4*>(kn + src) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    *reinterpret_cast<float4*>(qs + t * LDF + c) = in ? *reinterpret_cast<const float4*>(qn + src) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const __nv_bfloat16* src = qkv + (in ? (row0 + t) * C + g * DK + c : 0);
+    cp_async16(qt + t * LDN + c, src, in);
+    cp_async16(kt + t * LDN + c, src + (in ? G * DK : 0), in);
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
   if (CHANNEL) {
     for (int e = tid; e < L * DK; e += PREP_THREADS) {
       const int t = e / DK, i = e % DK;
@@ -128,27 +155,33 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
   } else if (tid < L) {
     cs[tid] = tid < count ? delta_log_decay(gates, row0 + tid, h, neg_a) : 0.0f;
   }
-  if (tid < L) betas[tid] = tid < count ? delta_beta(gates, row0 + tid, h) : 0.0f;
+  if (tid < L) {
+    const bool in = tid < count;
+    betas[tid] = in ? delta_beta(gates, row0 + tid, h) : 0.0f;
+    q_len_[tid] = in ? lengths[(row0 + tid) * 2 * G + g] : 0.0f;
+    k_len[tid] = in ? lengths[(row0 + tid) * 2 * G + G + g] : 0.0f;
+  }
   __syncthreads();
   // ---- running sums over the chunk
-  if (CHANNEL) {      // a thread per (channel, 16 tokens); then what the groups of 16 before have summed to
+  if (CHANNEL) {      // a thread per (channel, 16 or 32 tokens); then what the groups before have summed to
+    constexpr int PARTS = 4 * DK <= PREP_THREADS ? 4 : 2, LEN = L / PARTS;
     const int i = tid % DK, s = tid / DK;
     float run = 0.0f;
-    if (s < 4) {
-#pragma unroll
-      for (int t = 0; t < 16; ++t) {
-        run += cs[(s * 16 + t) * LDF + i];
-        cs[(s * 16 + t) * LDF + i] = run;
+    if (s < PARTS) {
+#pragma unroll 16
+      for (int t = 0; t < LEN; ++t) {
+        run += cs[(s * LEN + t) * LDF + i];
+        cs[(s * LEN + t) * LDF + i] = run;
       }
     }
     __syncthreads();
     float before = 0.0f;
-    if (s < 4)
-      for (int j = 0; j < s; ++j) before += cs[(j * 16 + 15) * LDF + i];
+    if (s < PARTS)
+      for (int j = 0; j < s; ++j) before += cs[(j * LEN + LEN - 1) * LDF + i];
     __syncthreads();
-    if (s > 0 && s < 4) {
-#pragma unroll
-      for (int t = 0; t < 16; ++t) cs[(s * 16 + t) * LDF + i] += before;
+    if (s > 0 && s < PARTS) {
+#pragma unroll 16
+      for (int t = 0; t < LEN; ++t) cs[(s * LEN + t) * LDF + i] += before;
     }
   } else if (warp == 0) {      // a lane takes two neighbours
     const float v0 = cs[2 * lane], v1 = cs[2 * lane + 1];
@@ -161,38 +194,53 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
     cs[2 * lane] = run - v1;
     cs[2 * lane + 1] = run;
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
 
   // ---- L and P, a warp per block of 16 x 16 pairs on or below the diagonal
   __nv_bfloat16* p_row = o.p + h * L;
   const long long p_stride = (long long)H * L;
-  if (warp < 10) {
-    const int a = warp < 1 ? 0 : (warp < 3 ? 1 : (warp < 6 ? 2 : 3)), b = warp - a * (a + 1) / 2;
+  for (int task = warp; task < 10; task += PREP_THREADS / 32) {
+    const int a = task < 1 ? 0 : (task < 3 ? 1 : (task < 6 ? 2 : 3)), b = task - a * (a + 1) / 2;
     const int t0 = 16 * a + gq;
+    const float* ref = cs + (16 * a - 1) * LDF;      // (CHANNEL, a > 0)
     bool one_by_one = false;
     if (CHANNEL && a == b) {
       float range = 0.0f;
-      for (int i = lane; i < DK; i += 32) range = fmaxf(range, (a ? cs[(16 * a - 1) * LDF + i] : 0.0f) - cs[(16 * a + 15) * LDF + i]);
+      for (int i = lane; i < DK; i += 32) range = fmaxf(range, (a ? ref[i] : 0.0f) - cs[(16 * a + 15) * LDF + i]);
       one_by_one = warp_max(range) > SAFE_RANGE;
     }
     float kk[2][4] = {}, qk[2][4] = {};
-    if (!one_by_one) {
+    if (!CHANNEL) {
+#pragma unroll
+      for (int s = 0; s < DK / 16; ++s) {
+        uint32_t ka[4], qa[4], kb[4];
+        const int at = (16 * a + (lane & 15)) * LDN + s * 16 + (lane >> 4) * 8;
+        ldmatrix_x4(ka, kt + at);
+        ldmatrix_x4(qa, qt + at);
+        ldmatrix_x4(kb, kt + (16 * b + (mid >> 1) * 8 + (lane & 7)) * LDN + s * 16 + (mid & 1) * 8);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          mma_bf16(kk[nt], ka, kb[nt * 2], kb[nt * 2 + 1]);
+          mma_bf16(qk[nt], qa, kb[nt * 2], kb[nt * 2 + 1]);
+        }
+      }
+    } else if (!one_by_one) {
 #pragma unroll 2
       for (int s = 0; s < DK / 16; ++s) {
         uint32_t kh[4], kl[4], qh[4], ql[4];
+        float2 r[2];
+#pragma unroll
+        for (int f = 0; f < 2; ++f)
+          r[f] = a ? *reinterpret_cast<const float2*>(ref + s * 16 + tq * 2 + f * 8) : make_float2(0.0f, 0.0f);
 #pragma unroll
         for (int f = 0; f < 4; ++f) {      // rows gq, gq + 8 of columns 2 tq, then of columns 2 tq + 8
           const int t = t0 + (f & 1) * 8, c = s * 16 + tq * 2 + (f >> 1) * 8;
-          float2 k2 = *reinterpret_cast<const float2*>(ks + t * LDF + c), q2 = *reinterpret_cast<const float2*>(qs + t * LDF + c);
-          if (CHANNEL) {
-            const float2 ct = *reinterpret_cast<const float2*>(cs + t * LDF + c);
-            const float2 r = a ? *reinterpret_cast<const float2*>(cs + (16 * a - 1) * LDF + c) : make_float2(0.0f, 0.0f);
-            const float e0 = expf(ct.x - r.x), e1 = expf(ct.y - r.y);
-            k2.x *= e0; k2.y *= e1;
-            q2.x *= e0; q2.y *= e1;
-          }
-          split2(k2.x, k2.y, kh[f], kl[f]);
-          split2(q2.x, q2.y, qh[f], ql[f]);
+          const float2 k2 = pair_of(kt + t * LDN + c), q2 = pair_of(qt + t * LDN + c);
+          const float2 ct = *reinterpret_cast<const float2*>(cs + t * LDF + c);
+          const float e0 = exp2f(ct.x - r[f >> 1].x), e1 = exp2f(ct.y - r[f >> 1].y);
+          split2(k2.x * e0, k2.y * e1, kh[f], kl[f]);
+          split2(q2.x * e0, q2.y * e1, qh[f], ql[f]);
         }
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
@@ -200,21 +248,11 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
 #pragma unroll
           for (int f = 0; f < 2; ++f) {
             const int j = 16 * b + nt * 8 + gq, c = s * 16 + tq * 2 + f * 8;
-            float2 k2 = *reinterpret_cast<const float2*>(ks + j * LDF + c);
-            if (CHANNEL) {
-              const float2 cj = *reinterpret_cast<const float2*>(cs + j * LDF + c);
-              const float2 r = a ? *reinterpret_cast<const float2*>(cs + (16 * a - 1) * LDF + c) : make_float2(0.0f, 0.0f);
-              k2.x *= expf(r.x - cj.x);
-              k2.y *= expf(r.y - cj.y);
-            }
-            split2(k2.x, k2.y, bh[f], bl[f]);
+            const float2 k2 = pair_of(kt + j * LDN + c), cj = *reinterpret_cast<const float2*>(cs + j * LDF + c);
+            split2(k2.x * exp2f(r[f].x - cj.x), k2.y * exp2f(r[f].y - cj.y), bh[f], bl[f]);
           }
-          mma_bf16(kk[nt], kh, bh[0], bh[1]);
-          mma_bf16(kk[nt], kh, bl[0], bl[1]);
-          mma_bf16(kk[nt], kl, bh[0], bh[1]);
-          mma_bf16(qk[nt], qh, bh[0], bh[1]);
-          mma_bf16(qk[nt], qh, bl[0], bl[1]);
-          mma_bf16(qk[nt], ql, bh[0], bh[1]);
+          mma_split(kk[nt], kh, kl, bh[0], bh[1], bl[0], bl[1]);
+          mma_split(qk[nt], qh, ql, bh[0], bh[1], bl[0], bl[1]);
         }
       }
     } else {
@@ -226,9 +264,9 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
           if (j > t) continue;
           float x = 0.0f, y = 0.0f;
           for (int i = 0; i < DK; ++i) {
-            const float f = ks[j * LDF + i] * expf(cs[t * LDF + i] - cs[j * LDF + i]);
-            x = fmaf(ks[t * LDF + i], f, x);
-            y = fmaf(qs[t * LDF + i], f, y);
+            const float f = __bfloat162float(kt[j * LDN + i]) * exp2f(cs[t * LDF + i] - cs[j * LDF + i]);
+            x = fmaf(__bfloat162float(kt[t * LDN + i]), f, x);
+            y = fmaf(__bfloat162float(qt[t * LDN + i]), f, y);
           }
           kk[nt][e] = x;
           qk[nt][e] = y;
@@ -242,9 +280,9 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
         float pv[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float f = CHANNEL ? 1.0f : (j + e <= t ? expf(cs[t] - cs[j + e]) : 0.0f);
-          pv[e] = j + e <= t ? qk[nt][r * 2 + e] * f : 0.0f;
-          Lm[t * LDT + j + e] = j + e < t ? betas[t] * kk[nt][r * 2 + e] * f : 0.0f;
+          const float f = j + e <= t ? (CHANNEL ? 1.0f : exp2f(cs[t] - cs[j + e])) * k_len[j + e] : 0.0f;
+          pv[e] = j + e <= t ? qk[nt][r * 2 + e] * q_len_[t] * f : 0.0f;
+          Lm[t * LDL + j + e] = j + e < t ? betas[t] * k_len[t] * kk[nt][r * 2 + e] * f : 0.0f;
         }
         if (t < count) {
           uint32_t hi, lo;
@@ -257,149 +295,207 @@ gated_delta_prepare_kernel(const float* __restrict__ qn, const float* __restrict
   }
   __syncthreads();
 
-  // ---- Q', K'' and (in place of k) K'; the decay over the chunk
-  for (int e = tid; e < L * (DK / 4); e += PREP_THREADS) {
-    const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-    float kd[4], qd[4], kend[4];
+  // ---- Q', K'' and (in place of k and q) K'; the decay over the chunk
+  for (int e = tid; e < L * (DK / 8); e += PREP_THREADS) {
+    const int t = e / (DK / 8), c = (e % (DK / 8)) * 8;
+    const uint4 k8 = *reinterpret_cast<const uint4*>(kt + t * LDN + c), q8 = *reinterpret_cast<const uint4*>(qt + t * LDN + c);
+    const __nv_bfloat16 *kp = reinterpret_cast<const __nv_bfloat16*>(&k8), *qp = reinterpret_cast<const __nv_bfloat16*>(&q8);
+    const float kn = k_len[t], qn = q_len_[t];
+    uint32_t hd[4], ld[4], hq[4], lq[4], he[4], le[4];
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
-      const float ct = CHANNEL ? cs[t * LDF + c + x] : cs[t], last = CHANNEL ? cs[(L - 1) * LDF + c + x] : cs[L - 1];
-      const float k = ks[t * LDF + c + x], f = expf(ct);
-      kd[x] = k * f;
-      qd[x] = qs[t * LDF + c + x] * f;
-      kend[x] = k * expf(last - ct);
+      const float2 k2 = pair_of(kp + 2 * x), q2 = pair_of(qp + 2 * x);
+      float f[2], last[2];
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const float ct = CHANNEL ? cs[t * LDF + c + 2 * x + y] : cs[t];
+        f[y] = exp2f(ct);
+        last[y] = exp2f((CHANNEL ? cs[(L - 1) * LDF + c + 2 * x + y] : cs[L - 1]) - ct);
+      }
+      split2(k2.x * kn * f[0], k2.y * kn * f[1], hd[x], ld[x]);
+      split2(q2.x * qn * f[0], q2.y * qn * f[1], hq[x], lq[x]);
+      split2(k2.x * kn * last[0], k2.y * kn * last[1], he[x], le[x]);
     }
-    *reinterpret_cast<float4*>(ks + t * LDF + c) = make_float4(kd[0], kd[1], kd[2], kd[3]);
+    *reinterpret_cast<uint4*>(kt + t * LDN + c) = make_uint4(hd[0], hd[1], hd[2], hd[3]);
+    *reinterpret_cast<uint4*>(qt + t * LDN + c) = make_uint4(ld[0], ld[1], ld[2], ld[3]);
     if (t < count) {
       const long long at = (row0 + t) * ((long long)H * DK) + h * DK + c;
-      uint2 hi, lo;
-      split2(qd[0], qd[1], hi.x, lo.x);
-      split2(qd[2], qd[3], hi.y, lo.y);
-      *reinterpret_cast<uint2*>(o.q + at) = hi;
-      *reinterpret_cast<uint2*>(o.q + o.hl + at) = lo;
-      split2(kend[0], kend[1], hi.x, lo.x);
-      split2(kend[2], kend[3], hi.y, lo.y);
-      *reinterpret_cast<uint2*>(o.k + at) = hi;
-      *reinterpret_cast<uint2*>(o.k + o.hl + at) = lo;
+      *reinterpret_cast<uint4*>(o.q + at) = make_uint4(hq[0], hq[1], hq[2], hq[3]);
+      *reinterpret_cast<uint4*>(o.q + o.hl + at) = make_uint4(lq[0], lq[1], lq[2], lq[3]);
+      *reinterpret_cast<uint4*>(o.k + at) = make_uint4(he[0], he[1], he[2], he[3]);
+      *reinterpret_cast<uint4*>(o.k + o.hl + at) = make_uint4(le[0], le[1], le[2], le[3]);
     }
   }
   if (tid < DK)
-    o.end[chunk_id(q_start, seq, chunk) * ((long long)H * DK) + h * DK + tid] = expf(CHANNEL ? cs[(L - 1) * LDF + tid] : cs[L - 1]);
-
-  // ---- (1 + L)^-1 in place: the blocks on the diagonal by substitution, a lane per column ...
-  if (warp < 4 && lane < 16) {
+    o.end[chunk_id(q_start, seq, chunk) * ((long long)H * DK) + h * DK + tid] = exp2f(CHANNEL ? cs[(L - 1) * LDF + tid] : cs[L - 1]);
+  // ---- (1 + L)^-1, the blocks on the diagonal by substitution, a lane per column ...
+  if (warp >= PREP_THREADS / 32 - 4 && lane < 16) {
+    const int a = warp - (PREP_THREADS / 32 - 4);
     float x[16];
-    const float* l = Lm + (16 * warp) * LDT + 16 * warp;
+    const float* l = Lm + (16 * a) * LDL + 16 * a;
+    const float beta = betas[16 * a + lane];
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
       float v = t == lane ? 1.0f : 0.0f;
 #pragma unroll
-      for (int s = 0; s < t; ++s) v = fmaf(-l[t * LDT + s], x[s], v);
+      for (int s = 0; s < t; ++s) v = fmaf(-l[t * LDL + s], x[s], v);
       x[t] = v;
     }
-    __syncwarp(0xffffu);
 #pragma unroll
-    for (int t = 0; t < 16; ++t) Lm[(16 * warp + t) * LDT + 16 * warp + lane] = x[t];
+    for (int t = 0; t < 16; ++t) {
+      const __nv_bfloat16 xh = __float2bfloat16_rn(x[t]), yh = __float2bfloat16_rn(x[t] * beta);
+      D[(a * 16 + t) * LDD + lane] = xh;
+      D[(64 + a * 16 + t) * LDD + lane] = __float2bfloat16_rn(x[t] - __bfloat162float(xh));
+      T[(16 * a + t) * LDP + 16 * a + lane] = yh;
+      T[(L + 16 * a + t) * LDP + 16 * a + lane] = __float2bfloat16_rn(x[t] * beta - __bfloat162float(yh));
+    }
   }
   __syncthreads();
-  // ... then row of blocks by row of blocks: T_ab = -T_aa sum_c L_ac T_cb
+  // the values of the first piece, into the place of the sums
+  auto load_values = [&](int v0) {
+    const int w8 = min(DK, dv - v0) / 8;
+    for (int e = tid; e < L * w8; e += PREP_THREADS) {
+      const int t = e / w8, c = (e % w8) * 8;
+      const bool in = t < count;
+      cp_async16(vt + t * LDN + c, qkv + (in ? (row0 + t) * C + 2LL * G * DK + (long long)h * dv + v0 + c : 0), in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load_values(0);
+  // ... then T = (1 + L)^-1 diag(beta) row of blocks by row of blocks, T_ab = -(1 + L)^-1_aa sum_c L_ac T_cb, a warp per
+  // block.  The sum is formed transposed: its accumulators then are the second product's operand as they lie.
   for (int a = 1; a < 4; ++a) {
-    float x[2];
+    if (warp < a) {
+      const int b = warp;
+      float xt[2][4] = {};      // [half of the rows t][...]: rows are the columns j of the block
+      for (int c = b; c < a; ++c) {
+        uint32_t th[4], tl[4];
+        const int at = (16 * c + (mid >> 1) * 8 + (lane & 7)) * LDP + 16 * b + (mid & 1) * 8;
+        ldmatrix_x4_trans(th, T + at);
+        ldmatrix_x4_trans(tl, T + L * LDP + at);
 #pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      const int e = tid + y * PREP_THREADS;
-      x[y] = 0.0f;
-      if (e < a * 256) {
-        const int t = (e >> 4) & 15, j = (e >> 8) * 16 + (e & 15);
-        for (int s = (j >> 4) * 16; s < 16 * a; ++s) x[y] = fmaf(Lm[(16 * a + t) * LDT + s], Lm[s * LDT + j], x[y]);
+        for (int nt = 0; nt < 2; ++nt) {
+          uint32_t bh[2], bl[2];
+#pragma unroll
+          for (int f = 0; f < 2; ++f) {
+            const float2 l2 = *reinterpret_cast<const float2*>(Lm + (16 * a + nt * 8 + gq) * LDL + 16 * c + tq * 2 + f * 8);
+            split2(l2.x, l2.y, bh[f], bl[f]);
+          }
+          mma_split(xt[nt], th, tl, bh[0], bh[1], bl[0], bl[1]);
+        }
       }
-    }
-    __syncthreads();
+      uint32_t dh[4], dl[4];
+      const int at = (a * 16 + (lane & 15)) * LDD + (lane >> 4) * 8;
+      ldmatrix_x4(dh, D + at);
+      ldmatrix_x4(dl, D + 64 * LDD + at);
 #pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      const int e = tid + y * PREP_THREADS;
-      if (e < a * 256) Lm[(16 * a + ((e >> 4) & 15)) * LDT + (e >> 8) * 16 + (e & 15)] = x[y];
-    }
-    __syncthreads();
+      for (int nj = 0; nj < 2; ++nj) {
+        uint32_t bh[2], bl[2];
+        split2(xt[0][nj * 2], xt[0][nj * 2 + 1], bh[0], bl[0]);
+        split2(xt[1][nj * 2], xt[1][nj * 2 + 1], bh[1], bl[1]);
+        float y[4] = {};
+        mma_split(y, dh, dl, bh[0], bh[1], bl[0], bl[1]);
 #pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      const int e = tid + y * PREP_THREADS;
-      x[y] = 0.0f;
-      if (e < a * 256) {
-        const int t = (e >> 4) & 15, j = (e >> 8) * 16 + (e & 15);
-#pragma unroll
-        for (int s = 0; s < 16; ++s) x[y] = fmaf(-Lm[(16 * a + t) * LDT + 16 * a + s], Lm[(16 * a + s) * LDT + j], x[y]);
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          split2(-y[r * 2], -y[r * 2 + 1], hi, lo);
+          const int dst = (16 * a + gq + r * 8) * LDP + 16 * b + nj * 8 + tq * 2;
+          *reinterpret_cast<uint32_t*>(T + dst) = hi;
+          *reinterpret_cast<uint32_t*>(T + L * LDP + dst) = lo;
+        }
       }
-    }
-    __syncthreads();
-#pragma unroll
-    for (int y = 0; y < 2; ++y) {
-      const int e = tid + y * PREP_THREADS;
-      if (e < a * 256) Lm[(16 * a + ((e >> 4) & 15)) * LDT + (e >> 8) * 16 + (e & 15)] = x[y];
     }
     __syncthreads();
   }
 
-  // ---- T K' and T V with T = (1 + L)^-1 diag(beta), a warp per 16 rows and 16 columns
-  const int tasks = 4 * (DK + dv) / 16;
-  for (int task = warp; task < tasks; task += PREP_THREADS / 32) {
-    const int m = 3 - (task & 3), n0 = (task >> 2) * 16;
-    const bool is_w = n0 < DK;
-    float acc[2][4] = {};
-    for (int kk = 0; kk <= m; ++kk) {
-      uint32_t th[4], tl[4];
+  // ---- T K' and T V: a warp has rows of blocks m0 and 3 - m0 (five blocks of T together) and every fourth 16 columns
+  const int m0 = warp & 1;
+  uint32_t th[2][4][4], tl[2][4][4];
 #pragma unroll
-      for (int f = 0; f < 4; ++f) {
-        const int t = 16 * m + gq + (f & 1) * 8, j = kk * 16 + tq * 2 + (f >> 1) * 8;
-        split2(Lm[t * LDT + j] * betas[j], Lm[t * LDT + j + 1] * betas[j + 1], th[f], tl[f]);
+  for (int y = 0; y < 2; ++y) {
+    const int m = y ? 3 - m0 : m0;
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk)
+      if (kk <= m) {
+        const int at = (16 * m + (lane & 15)) * LDP + kk * 16 + (lane >> 4) * 8;
+        ldmatrix_x4(th[y][kk], T + at);
+        ldmatrix_x4(tl[y][kk], T + L * LDP + at);
       }
+  }
+  for (int n0 = (warp >> 1) * 16; n0 < DK; n0 += 64) {
+    float acc[2][2][4] = {};
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        uint32_t bh[2], bl[2];
+    for (int kk = 0; kk < 4; ++kk) {
+      uint32_t bh[4], bl[4];
+      const int at = (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDN + n0 + (mid >> 1) * 8;
+      ldmatrix_x4_trans(bh, kt + at);
+      ldmatrix_x4_trans(bl, qt + at);
 #pragma unroll
-        for (int f = 0; f < 2; ++f) {
-          const int j = kk * 16 + tq * 2 + f * 8;
-          float v0, v1;
-          if (is_w) {
-            const int c = n0 + nt * 8 + gq;
-            v0 = ks[j * LDF + c];
-            v1 = ks[(j + 1) * LDF + c];
-          } else {
-            const long long src = (row0 + j) * ((long long)H * dv) + (long long)h * dv + (n0 - DK) + nt * 8 + gq;
-            v0 = j < count ? vn[src] : 0.0f;
-            v1 = j + 1 < count ? vn[src + (long long)H * dv] : 0.0f;
-          }
-          split2(v0, v1, bh[f], bl[f]);
+      for (int y = 0; y < 2; ++y)
+        if (kk <= (y ? 3 - m0 : m0)) {
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt)
+            mma_split(acc[y][nt], th[y][kk], tl[y][kk], bh[nt * 2], bh[nt * 2 + 1], bl[nt * 2], bl[nt * 2 + 1]);
         }
-        mma_bf16(acc[nt], th, bh[0], bh[1]);
-        mma_bf16(acc[nt], th, bl[0], bl[1]);
-        mma_bf16(acc[nt], tl, bh[0], bh[1]);
-      }
     }
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
+    for (int y = 0; y < 2; ++y)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const int t = 16 * m + gq + r * 8;
+        const int t = 16 * (y ? 3 - m0 : m0) + gq + r * 8;
         if (t >= count) continue;
-        if (is_w) {
-          __nv_bfloat16* dst = o.w + (row0 + t) * ((long long)H * DK) + h * DK + n0 + nt * 8 + tq * 2;
+        __nv_bfloat16* dst = o.w + (row0 + t) * ((long long)H * DK) + h * DK + n0 + tq * 2;
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
           uint32_t hi, lo;
-          split2(acc[nt][r * 2], acc[nt][r * 2 + 1], hi, lo);
-          *reinterpret_cast<uint32_t*>(dst) = hi;
-          *reinterpret_cast<uint32_t*>(dst + o.hl) = lo;
-        } else {
-          *reinterpret_cast<float2*>(o.u + (row0 + t) * ((long long)H * dv) + (long long)h * dv + (n0 - DK) + nt * 8 + tq * 2) =
-              make_float2(acc[nt][r * 2], acc[nt][r * 2 + 1]);
+          split2(acc[y][nt][r * 2], acc[y][nt][r * 2 + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(dst + nt * 8) = hi;
+          *reinterpret_cast<uint32_t*>(dst + o.hl + nt * 8) = lo;
         }
       }
+  }
+  for (int v0 = 0; v0 < dv; v0 += DK) {
+    if (v0 > 0) {
+      __syncthreads();      // the piece before this one has been read
+      load_values(v0);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int width = min(DK, dv - v0);
+    for (int n0 = (warp >> 1) * 16; n0 < width; n0 += 64) {
+      float acc[2][2][4] = {};
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        uint32_t vf[4];
+        ldmatrix_x4_trans(vf, vt + (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDN + n0 + (mid >> 1) * 8);
+#pragma unroll
+        for (int y = 0; y < 2; ++y)
+          if (kk <= (y ? 3 - m0 : m0)) {
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) {
+              mma_bf16(acc[y][nt], th[y][kk], vf[nt * 2], vf[nt * 2 + 1]);
+              mma_bf16(acc[y][nt], tl[y][kk], vf[nt * 2], vf[nt * 2 + 1]);
+            }
+          }
+      }
+#pragma unroll
+      for (int y = 0; y < 2; ++y)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = 16 * (y ? 3 - m0 : m0) + gq + r * 8;
+          if (t >= count) continue;
+          float* dst = o.u + (row0 + t) * ((long long)H * dv) + (long long)h * dv + v0 + n0 + tq * 2;
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt)
+            *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(acc[y][nt][r * 2], acc[y][nt][r * 2 + 1]);
+        }
+    }
   }
 }
 
 // ------------------------------------------------------------------------------------------- walk
 
-constexpr int WARPS = 4, THREADS = WARPS * 32;
-constexpr int LDN = DK + 8, LDP = L + 8;          // padded bfloat16 rows (conflict-free ldmatrix)
+constexpr int WARPS = 4;                          // warps that share the 64 tokens (and the state's row tiles)
 constexpr int MT_N = DK / 16;                     // row tiles of the state
 constexpr int MTW = (MT_N + WARPS - 1) / WARPS;   // of which a warp owns at most this many
 
@@ -409,12 +505,13 @@ struct WalkShared {
   static constexpr size_t BYTES = 2 * (size_t)(6 * L * LDN + 2 * L * LDP + 2 * DK * LDC + 2 * L * LDC) + 4 * DK;
 };
 
+// A block's warps: WARPS of them per group of 16 value columns.
 template <int PC>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(WARPS * 2 * PC)
 gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__ out, const int32_t* __restrict__ seq_slot,
                         const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_q_len, int H, int dv) {
   pdl_launch_dependents();
-  constexpr int LDC = WalkShared<PC>::LDC, NT = PC / 8;
+  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 2 * PC;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* Ws = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2][L][LDN]: rounded, rest (and so on below)
   __nv_bfloat16* Qs = Ws + 2 * L * LDN;
@@ -424,11 +521,14 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
   __nv_bfloat16* Us = Ss + 2 * DK * LDC;                               // [2][L][LDC]
   float* ends = reinterpret_cast<float*>(Us + 2 * L * LDC);            // [DK]
   pdl_wait();
-  const int col0 = blockIdx.x * PC, h = blockIdx.y, seq = blockIdx.z;
+  const int h = blockIdx.y, seq = blockIdx.z;
   const int q_len = seq_q_len[seq];
   if (q_len <= 0) return;
   const int q_start = seq_q_start[seq];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3, mid = lane >> 3;
+  const int warp = (threadIdx.x >> 5) % WARPS, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3, mid = lane >> 3;
+  const int own = (threadIdx.x >> 5) / WARPS * 16, col0 = blockIdx.x * PC + own;      // this warp's 16 columns
+  Ss += own;
+  Us += own;
   float* S_g = state + (((long long)seq_slot[seq] * H + h) * DK) * dv + col0;
   const int n_chunks = (q_len + L - 1) / L;
 
@@ -650,7 +750,7 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
 
 }  // namespace
 
-extern "C" int llm_gated_delta_prepare(const float* qn, const float* kn, const float* vn, const void* z, long long z_stride,
+extern "C" int llm_gated_delta_prepare(const void* qkv, const float* lengths, const void* z, long long z_stride,
                                        int z_dtype, const void* b, long long b_stride, int b_dtype, const float* a_log,
                                        const float* dt_bias, int channel, void* w, void* q, void* k, long long hl, void* p,
                                        long long p_hl, float* u, float* end, const int32_t* seq_q_start,
@@ -660,7 +760,7 @@ extern "C" int llm_gated_delta_prepare(const float* qn, const float* kn, const f
   LLM_HOST_CHECK(dk == DK && dv >= 16 && dv % 16 == 0 && kv_heads >= 1 && heads % kv_heads == 0, ERR_BAD_SIZE);
   LLM_HOST_CHECK(heads <= 65535 && n_seqs <= 65535 && hl % 8 == 0 && p_hl % 8 == 0, ERR_BAD_SIZE);
   LLM_HOST_CHECK((z_dtype == DT_F32 || z_dtype == DT_BF16) && (b_dtype == DT_F32 || b_dtype == DT_BF16), ERR_BAD_DTYPE);
-  LLM_HOST_CHECK((((uintptr_t)qn | (uintptr_t)kn | (uintptr_t)w | (uintptr_t)q | (uintptr_t)k | (uintptr_t)p | (uintptr_t)u |
+  LLM_HOST_CHECK((((uintptr_t)qkv | (uintptr_t)w | (uintptr_t)q | (uintptr_t)k | (uintptr_t)p | (uintptr_t)u |
                    (uintptr_t)end) & 15) == 0, ERR_BAD_ALIGN);
   const DeltaGates gates{z, z_stride, z_dtype, b, b_stride, b_dtype, a_log, dt_bias};
   const Tiles o{(__nv_bfloat16*)w, (__nv_bfloat16*)q, (__nv_bfloat16*)k, (__nv_bfloat16*)p, u, end, hl, p_hl};
@@ -675,8 +775,8 @@ extern "C" int llm_gated_delta_prepare(const float* qn, const float* kn, const f
         return launch_status();                                                                                         \
       configured = true;                                                                                                \
     }                                                                                                                   \
-    launch_kernel(gated_delta_prepare_kernel<CH>, grid, PREP_THREADS, smem, stream, qn, kn, vn, gates, o, seq_q_start,  \
-                  seq_q_len, heads, kv_heads, dv);                                                                      \
+    launch_kernel(gated_delta_prepare_kernel<CH>, grid, PREP_THREADS, smem, stream, (const __nv_bfloat16*)qkv, lengths,  \
+                  gates, o, seq_q_start, seq_q_len, heads, kv_heads, dv);                                               \
   } while (0)
   if (channel) GO(true); else GO(false);
 #undef GO
@@ -704,7 +804,7 @@ extern "C" int llm_gated_delta_walk(const void* w, const void* q, const void* k,
         return launch_status();                                                                                         \
       configured = true;                                                                                                \
     }                                                                                                                   \
-    launch_kernel(gated_delta_walk_kernel<PC>, grid, THREADS, smem, stream, in, state, out, seq_slot, seq_q_start,      \
+    launch_kernel(gated_delta_walk_kernel<PC>, grid, WARPS * 2 * PC, smem, stream, in, state, out, seq_slot, seq_q_start,      \
                   seq_q_len, heads, dv);                                                                                \
   } while (0)
   if (columns == 16) GO(16); else GO(32);

@@ -167,34 +167,33 @@ extern "C" int llm_mamba2_finish(const float* scanned, const float* xc, const fl
 }
 
 // The projection rows [x | B | C] of each request's last taps - 1 positions go into its ring (entry position %
-// taps).  Grid (row, slice of channels).
+// taps).  Grid (request x kept position, slice of channels).
 template <typename T>
 __global__ void __launch_bounds__(256)
 mamba2_ring_write_kernel(const T* __restrict__ u, long long u_stride, float* __restrict__ ring, int taps, int C,
-                         const int32_t* __restrict__ positions, const int32_t* __restrict__ row_seq,
-                         const int32_t* __restrict__ seq_slot, const int32_t* __restrict__ seq_kv_len) {
+                         const int32_t* __restrict__ seq_slot, const int32_t* __restrict__ seq_q_start,
+                         const int32_t* __restrict__ seq_q_len, const int32_t* __restrict__ seq_kv_len) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x;
-  const int seq = row_seq[t], p = positions[t];
-  const int end = seq_kv_len[seq] > 0 ? seq_kv_len[seq] : p + 1;   // an idle row stands for itself
-  if (p < end - (taps - 1)) return;
+  const int seq = blockIdx.x / (taps - 1), back = blockIdx.x % (taps - 1) + 1;      // the request's last, last but one, ...
+  if (back > seq_q_len[seq]) return;
+  const int t = seq_q_start[seq] + seq_q_len[seq] - back, p = seq_kv_len[seq] - back;
   float* dst = ring + ((long long)seq_slot[seq] * taps + (p % taps)) * C;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
     dst[c] = to_float(u[(long long)t * u_stride + c]);
 }
 
 extern "C" int llm_mamba2_ring_write(const void* u, int dtype, long long u_stride, float* ring, int taps, int channels,
-                                     const int32_t* positions, const int32_t* row_seq, const int32_t* seq_slot,
-                                     const int32_t* seq_kv_len, int n_tokens, cudaStream_t stream) {
-  if (n_tokens <= 0 || taps <= 1) return 0;
-  const dim3 grid(n_tokens, n_tokens >= 64 ? 1 : (channels + 1023) / 1024);
+                                     const int32_t* seq_slot, const int32_t* seq_q_start, const int32_t* seq_q_len,
+                                     const int32_t* seq_kv_len, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0 || taps <= 1) return 0;
+  const dim3 grid(n_seqs * (taps - 1), (channels + 1023) / 1024);
   if (dtype == DT_F32)
     launch_kernel(mamba2_ring_write_kernel<float>, grid, 256, 0, stream, (const float*)u, u_stride, ring, taps, channels,
-                  positions, row_seq, seq_slot, seq_kv_len);
+                  seq_slot, seq_q_start, seq_q_len, seq_kv_len);
   else if (dtype == DT_BF16)
     launch_kernel(mamba2_ring_write_kernel<__nv_bfloat16>, grid, 256, 0, stream, (const __nv_bfloat16*)u, u_stride, ring,
-                  taps, channels, positions, row_seq, seq_slot, seq_kv_len);
+                  taps, channels, seq_slot, seq_q_start, seq_q_len, seq_kv_len);
   else
     return ERR_BAD_DTYPE;
   return launch_status();

@@ -4,7 +4,7 @@ distance over the paged cache (key and value heads may differ in size)."""
 
 from __future__ import annotations
 
-from ctypes import c_float, c_int, c_longlong, c_void_p
+from ctypes import byref, c_float, c_int, c_longlong, c_void_p
 from typing import Optional
 
 import torch
@@ -21,7 +21,7 @@ def lib():
         l = build.load_library("biased_attention.cu")
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
         l.llm_conv_norm_cache.argtypes = [P, I, L, P, I, P, P, P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, I, I, F, F,
-                                          I, I, P, I, I, P]
+                                          I, I, P, I, I, I, P, P]
         l.llm_conv_ring_write.argtypes = [P, I, L, P, I, I, P, P, P, P, I, P]
         l.llm_biased_attention.argtypes = [P, P, I, L, P, P, P, L, I, I, I, I, I, P, I, P, P, I, I, F, I, F, F, I, P, P, L, P]
         for name in ("llm_conv_norm_cache", "llm_conv_ring_write", "llm_biased_attention"):
@@ -33,11 +33,14 @@ def lib():
 def conv_norm_cache(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, q_norm_w: torch.Tensor,
                     k_norm_w: torch.Tensor, q_out: torch.Tensor, cache: CacheView, q_heads: int, eps: float,
                     temp_coef: float, temp_every: int, write_cache: bool, inv_freq: Optional[torch.Tensor] = None,
-                    rot_dims: int = 0, halves: bool = False) -> None:
+                    rot_dims: int = 0, halves: bool = False, write_ring: bool = False) -> bool:
     """u [rows, q | k | v channels] (may be a column view) -> causal convolution over time with
     `conv_w` [channels, taps] (history before the step from `ring`), RMS norm of all q channels and
     of all k channels, the position factor on q; with `inv_freq` the first `rot_dims` entries of every q and
-    k head turned by position (neighbouring pairs, or `halves`); q to `q_out`, k and v into the cache."""
+    k head turned by position (neighbouring pairs, or `halves`); q to `q_out`, k and v into the cache.  With
+    `write_ring` (steps of one token per request only) the kernel may also put the token's rows into the ring;
+    returns whether it has."""
+    written = c_int(0)
     _dev(u, conv_w, ring, q_norm_w, k_norm_w, q_out, inv_freq)
     _check(lib().llm_conv_norm_cache(
         u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(),
@@ -45,14 +48,16 @@ def conv_norm_cache(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tens
         cache.block_table.data_ptr(), cache.page_stride, cache.table_stride, cache.page_tokens, cache.kv_heads,
         cache.head_dim, cache.v_dim, ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
         ctx.seq_q_start.data_ptr(), ctx.n_tokens, q_heads, float(eps), float(temp_coef), int(temp_every),
-        1 if write_cache else 0, _ptr(inv_freq), int(rot_dims), 1 if halves else 0, ctx.stream), "conv_norm_cache")
+        1 if write_cache else 0, _ptr(inv_freq), int(rot_dims), 1 if halves else 0,
+        1 if write_ring else 0, byref(written), ctx.stream), "conv_norm_cache")
+    return bool(written.value)
 
 
 def conv_ring_write(ctx, u: torch.Tensor, ring: torch.Tensor, taps: int, channels: int) -> None:
     _dev(u, ring)
     _check(lib().llm_conv_ring_write(u.data_ptr(), dtype_code(u.dtype), u.stride(0), ring.data_ptr(), taps, channels,
-                                     ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
-                                     ctx.seq_kv_len.data_ptr(), ctx.n_tokens, ctx.stream), "conv_ring_write")
+                                     ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.seq_q_len.data_ptr(),
+                                     ctx.seq_kv_len.data_ptr(), ctx.n_seqs, ctx.stream), "conv_ring_write")
 
 
 def attention(ctx, q: torch.Tensor, out: torch.Tensor, cache: CacheView, bias: Optional[torch.Tensor], q_heads: int,

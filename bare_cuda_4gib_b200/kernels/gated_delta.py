@@ -9,7 +9,7 @@ from typing import Optional
 import torch
 
 from . import build
-from .lib import _check, _dev, dtype_code
+from .lib import _check, _dev, _ptr, dtype_code
 
 MAX_KEY_DIM = 1024
 STEP_MAX_SHARED = 160 * 1024
@@ -21,7 +21,7 @@ def lib():
     if _lib is None:
         l = build.load_library("gated_delta.cu")
         P, I, L, F = c_void_p, c_int, c_longlong, c_float
-        l.llm_gated_delta_operands.argtypes = [P, I, L, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, F, F, P]
+        l.llm_gated_delta_operands.argtypes = [P, I, L, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, F, F, P, P, P]
         l.llm_gated_delta_scan.argtypes = [P, P, P, P, L, I, P, L, I, P, P, I, P, P, P, P, P, I, I, I, I, I, P]
         l.llm_gated_delta_step.argtypes = [P, I, L, P, I, P, P, L, I, P, L, I, P, P, I, P, P, L, I, I, P, P, L, P, P, P, I, I, I,
                                            I, I, I, F, F, F, P]
@@ -58,16 +58,21 @@ def _floats(what: str, *tensors: Optional[torch.Tensor]) -> None:
             raise TypeError(f"gated delta {what}: constants, states and operands must be contiguous float32")
 
 
-def operands(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, qn: torch.Tensor, kn: torch.Tensor,
-             vn: torch.Tensor, kv_heads: int, dk: int, heads: int, dv: int, unit_eps: float) -> None:
+def operands(ctx, u: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, qn, kn, vn, kv_heads: int, dk: int,
+             heads: int, dv: int, unit_eps: float, compact: Optional[torch.Tensor] = None,
+             lengths: Optional[torch.Tensor] = None) -> None:
     """u [rows, q | k | v | ...]: the convolution (history before the step from `ring`) and silu; qn, kn [rows,
-    kv_heads * dk] the unit vectors (q also / sqrt(dk)), vn [rows, heads * dv].  All float32."""
-    _floats("operands", conv_w, ring, qn, kn, vn)
+    kv_heads * dk] the unit vectors (q also / sqrt(dk)), vn [rows, heads * dv].  All float32.  With `compact`
+    (bfloat16 [rows, q | k | v]) these are left out: the activations go there, and to `lengths` (float32 [rows,
+    2 * kv_heads], the q heads first) the factors that make the unit vectors of the rounded q and k heads."""
+    _floats("operands", conv_w, ring, qn, kn, vn, lengths)
+    if compact is not None and (compact.dtype != torch.bfloat16 or not compact.is_contiguous() or lengths is None):
+        raise TypeError("gated delta operands: the compact form is contiguous bfloat16 with float32 factors beside it")
     _check(lib().llm_gated_delta_operands(
-        u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(), qn.data_ptr(),
-        kn.data_ptr(), vn.data_ptr(), ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
-        ctx.seq_q_start.data_ptr(), ctx.n_tokens, kv_heads, dk, heads, dv, float(unit_eps), dk ** -0.5, ctx.stream),
-        "gated_delta_operands")
+        u.data_ptr(), dtype_code(u.dtype), u.stride(0), conv_w.data_ptr(), conv_w.shape[1], ring.data_ptr(), _ptr(qn),
+        _ptr(kn), _ptr(vn), ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
+        ctx.seq_q_start.data_ptr(), ctx.n_tokens, kv_heads, dk, heads, dv, float(unit_eps), dk ** -0.5, _ptr(compact),
+        _ptr(lengths), ctx.stream), "gated_delta_operands")
 
 
 def scan(ctx, qn: torch.Tensor, kn: torch.Tensor, vn: torch.Tensor, gates: Gates, state: torch.Tensor, out: torch.Tensor,
@@ -126,18 +131,21 @@ def chunked_lib(dk: int):
     if l is None:
         l = build.load_library("gated_delta_chunked.cu", (f"-DGD_DK={dk}",))
         P, I, L = c_void_p, c_int, c_longlong
-        l.llm_gated_delta_prepare.argtypes = [P, P, P, P, L, I, P, L, I, P, P, I, P, P, P, L, P, L, P, P, P, P, I, I, I, I, I, I, P]
+        l.llm_gated_delta_prepare.argtypes = [P, P, P, L, I, P, L, I, P, P, I, P, P, P, L, P, L, P, P, P, P, I, I, I, I, I, I, P]
         l.llm_gated_delta_walk.argtypes = [P, P, P, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P]
         l.llm_gated_delta_prepare.restype = l.llm_gated_delta_walk.restype = c_int
         _chunked_libs[dk] = l
     return l
 
 
-def chunked(ctx, qn: torch.Tensor, kn: torch.Tensor, vn: torch.Tensor, gates: Gates, state: torch.Tensor, out: torch.Tensor,
+def chunked(ctx, compact: torch.Tensor, lengths: torch.Tensor, gates: Gates, state: torch.Tensor, out: torch.Tensor,
             heads: int, kv_heads: int, dk: int, dv: int, columns: int = 0) -> None:
-    """What `scan` does, in chunks of 64 tokens on the tensor cores: two kernels, one over all chunks side by side
-    for everything that does not depend on the state, one that walks every request's chunks in order."""
-    _floats("chunked", qn, kn, vn, state, out)
+    """What `scan` does, in chunks of 64 tokens on the tensor cores, from the compact operands: two kernels, one over
+    all chunks side by side for everything that does not depend on the state, one that walks every request's
+    chunks in order."""
+    _floats("chunked", lengths, state, out)
+    if compact.dtype != torch.bfloat16 or not compact.is_contiguous():
+        raise TypeError("gated delta chunked: the operands must be contiguous bfloat16")
     columns = columns or chunked_columns(heads, dv)
     n = ctx.n_tokens
     tiles = ctx.ws.get("delta_tiles", (6, n, heads * dk), torch.bfloat16, max_lead=6)      # (W, Q', K'') x (rounded, rest)
@@ -150,7 +158,7 @@ def chunked(ctx, qn: torch.Tensor, kn: torch.Tensor, vn: torch.Tensor, gates: Ga
     at = [tiles.data_ptr() + 2 * plane * i for i in range(6)]
     where = (at[0], at[1], at[2], 3 * plane, pairs.data_ptr(), pairs.stride(0), u.data_ptr(), end.data_ptr())
     _check(l.llm_gated_delta_prepare(
-        qn.data_ptr(), kn.data_ptr(), vn.data_ptr(), *gates.arguments(), *where, ctx.seq_q_start.data_ptr(),
+        compact.data_ptr(), lengths.data_ptr(), *gates.arguments(), *where, ctx.seq_q_start.data_ptr(),
         ctx.seq_q_len.data_ptr(), ctx.n_seqs, int(ctx.max_q_len), heads, kv_heads, dk, dv, ctx.stream), "gated_delta_prepare")
     _check(l.llm_gated_delta_walk(
         *where, state.data_ptr(), out.data_ptr(), ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(),

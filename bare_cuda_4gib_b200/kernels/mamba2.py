@@ -72,8 +72,8 @@ def ring_write(ctx, u: torch.Tensor, ring: torch.Tensor, taps: int, channels: in
     [slots, taps, channels], entry position % taps."""
     _dev(u, ring)
     _check(lib().llm_mamba2_ring_write(u.data_ptr(), dtype_code(u.dtype), u.stride(0), ring.data_ptr(), taps, channels,
-                                       ctx.positions.data_ptr(), ctx.row_seq.data_ptr(), ctx.seq_slot.data_ptr(),
-                                       ctx.seq_kv_len.data_ptr(), ctx.n_tokens, ctx.stream), "mamba2_ring_write")
+                                       ctx.seq_slot.data_ptr(), ctx.seq_q_start.data_ptr(), ctx.seq_q_len.data_ptr(),
+                                       ctx.seq_kv_len.data_ptr(), ctx.n_seqs, ctx.stream), "mamba2_ring_write")
 
 
 STEP_MAX_SHARED = 160 * 1024

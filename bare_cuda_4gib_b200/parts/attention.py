@@ -358,9 +358,10 @@ class GeneralAttention(Part):
         q = ctx.ws.get("q", (n, self.qd), ctx.dtype)
         shared = ctx.ws.get("mixed_values", (n, self.vd), torch.float32) if self.v_mix else None
         if self.taps:
-            BA.conv_norm_cache(ctx, u, self.conv_w, call.state, self.q_norm, self.k_norm, q, call.cache, self.heads, self.eps,
-                               0.0, 1, call.writes_cache, self.inv_freq, self.rot_dims, self.halves)
-            if call.writes_cache:
+            kept = BA.conv_norm_cache(ctx, u, self.conv_w, call.state, self.q_norm, self.k_norm, q, call.cache, self.heads,
+                                      self.eps, 0.0, 1, call.writes_cache, self.inv_freq, self.rot_dims, self.halves,
+                                      write_ring=call.writes_cache and ctx.max_q_len == 1)
+            if call.writes_cache and not kept:
                 BA.conv_ring_write(ctx, u, call.state, self.taps, self.qd + self.kd + self.vd)
         else:
             self._prepare_heads(ctx, call, u, q, shared)

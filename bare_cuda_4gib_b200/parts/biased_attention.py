@@ -104,9 +104,10 @@ class BiasedAttention(BranchMixer):
     def inner(self, ctx, cache, state, writes, u, out, out_scale) -> None:
         n, p = ctx.n_tokens, self.params
         q = ctx.ws.get("biased_q", (n, self.qd), ctx.dtype)
-        BA.conv_norm_cache(ctx, u, self.conv_w, state, self.q_norm_w, self.k_norm_w, q, cache, self.heads,
-                           float(p["eps"]), float(p["temp_coef"]), int(p["temp_every"]), writes)
-        if writes:
+        kept = BA.conv_norm_cache(ctx, u, self.conv_w, state, self.q_norm_w, self.k_norm_w, q, cache, self.heads,
+                                  float(p["eps"]), float(p["temp_coef"]), int(p["temp_every"]), writes,
+                                  write_ring=writes and ctx.max_q_len == 1)
+        if writes and not kept:
             BA.conv_ring_write(ctx, u, state, self.taps, self.qd + self.kd + self.vd)
         window = int(self.window) if self.window else 0
         if self.fast is not None and ctx.use_fast_attention:

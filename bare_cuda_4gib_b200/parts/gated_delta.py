@@ -16,8 +16,8 @@ of the mixer's input, and projected.  Options:
 One product makes everything that reads h; with low ranks a second one multiplies both of them by their upper
 halves ([a2 0; 0 g2] over [a1 h | g1 h], float32 results).  A request keeps S as a float32 state and the
 convolution's last inputs as a second one (a ring of `taps` entries by position).  Steps of one token per request
-run one kernel with a block per (request, head); other steps prepare float32 operands, walk the state, and norm
-and gate.  The walk goes token by token, or in bfloat16 steps with a portion of `kernels.gated_delta.
+run one kernel with a block per (request, head); other steps prepare operands, walk the state, and norm
+and gate.  The walk goes token by token over float32 operands, or in bfloat16 steps with a portion of `kernels.gated_delta.
 CHUNKED_MIN_TOKENS` or more (sizes that are multiples of 16) in chunks on the tensor cores.
 
 params: `hidden`, `heads`, `kv_heads`, `dim`, `vdim`, `taps`, `decay`, `gate`, `rank` (None: from the file),
@@ -140,15 +140,21 @@ class GatedDelta(Part):
             GD.step(ctx, u, self.conv_w, ring, gates, state, gate, self.gate_kind, self.norm_w, out, H, G, dk, dv,
                     self.unit_eps, self.eps, call.writes_cache)
             return self.o.forward(ctx, out, n, f32, "mixer_out", allow_partials=True)
-        qn, kn = ctx.ws.get("delta_q", (n, self.kd), f32), ctx.ws.get("delta_k", (n, self.kd), f32)
-        vn = ctx.ws.get("delta_v", (n, self.vd), f32)
         scanned = ctx.ws.get("delta_scan", (n, self.vd), f32)
-        GD.operands(ctx, u, self.conv_w, ring, qn, kn, vn, G, dk, H, dv, self.unit_eps)
+        chunked = self.chunked and ctx.max_q_len >= GD.CHUNKED_MIN_TOKENS and ctx.use_fast_attention
+        if chunked:
+            compact = ctx.ws.get("delta_compact", (n, self.conv_channels), torch.bfloat16)
+            lengths = ctx.ws.get("delta_lengths", (n, 2 * G), f32)
+            GD.operands(ctx, u, self.conv_w, ring, None, None, None, G, dk, H, dv, self.unit_eps, compact, lengths)
+        else:
+            qn, kn = ctx.ws.get("delta_q", (n, self.kd), f32), ctx.ws.get("delta_k", (n, self.kd), f32)
+            vn = ctx.ws.get("delta_v", (n, self.vd), f32)
+            GD.operands(ctx, u, self.conv_w, ring, qn, kn, vn, G, dk, H, dv, self.unit_eps)
         if call.writes_cache:
             from ..kernels import mamba2 as MK
             MK.ring_write(ctx, u[:, : self.conv_channels], ring, self.taps, self.conv_channels)
-        if self.chunked and ctx.max_q_len >= GD.CHUNKED_MIN_TOKENS and ctx.use_fast_attention:
-            GD.chunked(ctx, qn, kn, vn, gates, state, scanned, H, G, dk, dv)
+        if chunked:
+            GD.chunked(ctx, compact, lengths, gates, state, scanned, H, G, dk, dv)
         else:
             GD.scan(ctx, qn, kn, vn, gates, state, scanned, H, G, dk, dv)
         LA.gated_group_norm(scanned, gate, self.norm_w, out, n, dv, self.gate_kind, self.eps, 1.0, ctx.stream)

@@ -53,11 +53,12 @@ def _ctx(lengths, dtype=torch.bfloat16, slots=None):
 
 
 def _inputs(n, heads, kv_heads, dk, dv, channel, seed, strength=0.0):
-    """Unit keys and queries, values, and gates; `strength` shifts the decays' logarithms towards faster decay."""
+    """Keys, queries and values that bfloat16 holds exactly, and gates; `strength` shifts the decays' logarithms
+    towards faster decay."""
     g = torch.Generator().manual_seed(seed)
     r = lambda *s: torch.randn(*s, generator=g)
-    q, k = P.unit_vector(r(n, kv_heads, dk)) * dk ** -0.5, P.unit_vector(r(n, kv_heads, dk))
-    v, b = r(n, heads, dv), 2.0 * r(n, heads)
+    q, k, v = (r(n, h, d).to(torch.bfloat16).double() for h, d in ((kv_heads, dk), (kv_heads, dk), (heads, dv)))
+    b = 2.0 * r(n, heads)
     zd = heads * dk if channel else heads
     z, a_log, dt_bias = r(n, zd), 0.5 * r(heads) + strength - 1.0, r(zd)
     return q, k, v, z, b, a_log, dt_bias
@@ -95,14 +96,17 @@ def _run(lengths, sizes, channel, seed, form, strength=0.0):
     ctx = _ctx(lengths)
     q, k, v, z, b, a_log, dt_bias = _inputs(n, heads, kv_heads, dk, dv, channel, seed, strength)
     start = 0.3 * torch.randn(len(lengths) + 1, heads, dk, dv, generator=torch.Generator().manual_seed(seed + 1))
-    want, want_state = _want(q, k, v, z, b, a_log, dt_bias, channel, lengths, ctx.slots, start)
+    qn, kn = P.unit_vector(q) * dk ** -0.5, P.unit_vector(k)
+    want, want_state = _want(qn, kn, v, z, b, a_log, dt_bias, channel, lengths, ctx.slots, start)
     c = lambda t: t.reshape(t.shape[0], -1).float().cuda().contiguous()
     state, out = start.cuda(), torch.full((n, heads * dv), float("nan"), **F32)
     gates = GD.Gates(c(z), c(b), a_log.cuda(), dt_bias.cuda(), channel)
     if form == "scan":
-        GD.scan(ctx, c(q), c(k), c(v), gates, state, out, heads, kv_heads, dk, dv)
+        GD.scan(ctx, c(qn), c(kn), c(v), gates, state, out, heads, kv_heads, dk, dv)
     else:
-        GD.chunked(ctx, c(q), c(k), c(v), gates, state, out, heads, kv_heads, dk, dv, form)
+        compact = torch.cat([c(q), c(k), c(v)], 1).to(torch.bfloat16).contiguous()
+        factors = torch.cat([dk ** -0.5 / torch.sqrt((q * q).sum(-1) + 1e-6), 1.0 / torch.sqrt((k * k).sum(-1) + 1e-6)], 1)
+        GD.chunked(ctx, compact, c(factors), gates, state, out, heads, kv_heads, dk, dv, form)
     torch.cuda.synchronize()
     assert torch.equal(state[-1].cpu(), start[-1])              # a slot that no request of the step holds
     scale, sscale = float(want.abs().max()), float(want_state[:-1].abs().max())
@@ -138,7 +142,7 @@ def test_chunks_with_decays_that_leave_nothing(channel, strength):
     """Decays so strong that the factors against a common token leave float32's range inside 16 tokens for some
     channels, while others keep most of what they hold."""
     err, serr = _run([130, 20], (4, 2, 32, 32), channel, 7, 16, strength)
-    assert err < 3e-4 and serr < 3e-4, (err, serr)
+    assert err < 2e-3 and serr < 2e-3, (err, serr)      # (a difference of two sums of large logarithms has fewer digits)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -196,6 +200,98 @@ def test_operands_against_plain_pieces(taps):
     assert H.row_error(qn, (P.unit_vector(y[:, :kd].view(n, kv_heads, dk)) * dk ** -0.5).reshape(n, kd)) < 1e-5
     assert H.row_error(kn, P.unit_vector(y[:, kd: 2 * kd].view(n, kv_heads, dk)).reshape(n, kd)) < 1e-5
     assert H.row_error(vn, y[:, 2 * kd:]) < 1e-5
+
+
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 6])
+@pytest.mark.parametrize("heads,kv_heads,dk,dv", [(4, 2, 16, 20), (2, 2, 128, 64), (3, 1, 48, 16), (6, 3, 32, 36), (2, 1, 64, 130)])
+def test_compact_operands_over_two_steps(heads, kv_heads, dk, dv, taps):
+    """Activations and unit factors of requests that go on from a ring, cut inside the convolution's reach, in the
+    form that walks rows and in the one with a block per token."""
+    from bare_cuda_4gib_b200.kernels import gated_delta as GD, mamba2 as MK
+    kd, C = kv_heads * dk, 2 * kv_heads * dk + heads * dv
+    cuts, total = ([19, 1, 3, 40], [2, 5, 1, 20]), [21, 6, 4, 60]
+    g = torch.Generator().manual_seed(taps)
+    u = [torch.randn(n, C + 8, generator=g).to(torch.bfloat16) for n in total]
+    w = torch.randn(C, taps, generator=g)
+    want = [P.silu(P.short_convolution(x[:, :C].double(), w.double())).to(torch.bfloat16).double() for x in u]
+    ring = torch.full((5, taps, C), float("nan"), **F32)
+    done = [0] * 4
+    for cut in cuts:
+        ctx = _ctx(cut)
+        ctx.positions = torch.cat([torch.arange(d, d + n) for d, n in zip(done, cut)]).to(torch.int32).cuda()
+        ctx.seq_kv_len = torch.tensor([d + n for d, n in zip(done, cut)], dtype=torch.int32, device="cuda")
+        rows = torch.cat([x[d: d + n] for x, d, n in zip(u, done, cut)]).cuda()
+        compact = torch.full((sum(cut), C), float("nan"), dtype=torch.bfloat16, device="cuda")
+        factors = torch.full((sum(cut), 2 * kv_heads), float("nan"), **F32)
+        GD.operands(ctx, rows, w.cuda(), ring, None, None, None, kv_heads, dk, heads, dv, 1e-6, compact, factors)
+        MK.ring_write(ctx, rows[:, :C], ring, taps, C)
+        y = torch.cat([x[d: d + n] for x, d, n in zip(want, done, cut)])
+        got = compact.double().cpu()
+        assert float((got - y).abs().max()) < 2e-2 * float(y.abs().max()) and float((got != y).double().mean()) < 0.02
+        heads_ = got[:, : 2 * kd].view(sum(cut), 2 * kv_heads, dk)
+        f = 1.0 / torch.sqrt((heads_ * heads_).sum(-1) + 1e-6)
+        f[:, :kv_heads] *= dk ** -0.5
+        assert H.row_error(factors, f) < 1e-5
+        done = [d + n for d, n in zip(done, cut)]
+
+
+@pytest.mark.parametrize("taps", [1, 2, 4, 6])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("heads,kv_heads,dk,dv,rot", [(4, 2, 16, 24, 8), (2, 1, 128, 128, 128), (16, 4, 128, 64, 32), (3, 3, 10, 7, 6),
+                                                      (32, 8, 128, 128, 64)])
+def test_convolution_norm_rotation_and_cache(heads, kv_heads, dk, dv, rot, dtype, taps):
+    """What stands between the projection and the scores, over three steps of requests that go on from their rings,
+    the last one of single tokens: queries, and keys and values in their pages."""
+    from bare_cuda_4gib_b200.kernels import biased_attention as BA
+    from bare_cuda_4gib_b200.kernels.lib import CacheView
+    qd, kd, vd, page, eps, base = heads * dk, kv_heads * dk, kv_heads * dv, 16, 1e-5, 300.0
+    C, hist = qd + kd + vd, max(taps - 1, 1)
+    if (heads, dk) == (4, 16):      # long portions: a block of the kernel walks several rows
+        cuts = ([700, 1, 400], [2, 5, 30], [1, 1, 1])
+    else:
+        cuts = ([19, 1, 7], [2, 5, 30], [1, 1, 1])
+    total = [sum(c[i] for c in cuts) for i in range(3)]
+    g = torch.Generator().manual_seed(taps)
+    u = [torch.randn(n, C + 8, generator=g).to(dtype) for n in total]
+    w, qw, kw = torch.randn(C, taps, generator=g), 1 + 0.2 * torch.randn(qd, generator=g), 1 + 0.2 * torch.randn(kd, generator=g)
+    want = []
+    for x, n in zip(u, total):
+        y = P.short_convolution(x[:, :C].double(), w.double())
+        pos = torch.arange(n)
+        q = P.turn_neighbours((P.unit_rms(y[:, :qd], eps) * qw.double()).view(n, heads, dk), pos, rot, base)
+        k = P.turn_neighbours((P.unit_rms(y[:, qd: qd + kd], eps) * kw.double()).view(n, kv_heads, dk), pos, rot, base)
+        want.append((q.reshape(n, qd), k, y[:, qd + kd:].view(n, kv_heads, dv)))
+    per = kv_heads * page * (dk + dv)
+    blocks = max(total) // page + 1
+    pool = torch.full((3 * blocks, per), float("nan"), dtype=dtype, device="cuda")
+    table = torch.randperm(3 * blocks, generator=g).view(3, blocks).to(torch.int32).cuda()
+    cache = CacheView(pool.data_ptr(), pool.data_ptr() + kv_heads * page * dk * pool.element_size(), table, per, blocks, page, kv_heads,
+                      dk, dtype, v_dim=dv)
+    ring = torch.zeros(4, hist, C, **F32)
+    freq = torch.tensor([base ** (-2.0 * i / rot) for i in range(rot // 2)], **F32)
+    done = [0] * 3
+    tol = 2e-5 if dtype == torch.float32 else 2e-2
+    for cut in cuts:
+        ctx = _ctx(cut, dtype)
+        ctx.positions = torch.cat([torch.arange(d, d + n) for d, n in zip(done, cut)]).to(torch.int32).cuda()
+        ctx.seq_kv_len = torch.tensor([d + n for d, n in zip(done, cut)], dtype=torch.int32, device="cuda")
+        rows = torch.cat([x[d: d + n] for x, d, n in zip(u, done, cut)]).cuda()
+        q_out = torch.full((sum(cut), qd), float("nan"), dtype=dtype, device="cuda")
+        kept = BA.conv_norm_cache(ctx, rows, w.cuda(), ring, qw.cuda(), kw.cuda(), q_out, cache, heads, eps, 0.0, 1, True, freq, rot,
+                                  False, write_ring=max(cut) == 1)
+        if not kept:
+            BA.conv_ring_write(ctx, rows, ring, taps, C)
+        assert H.row_error(q_out, torch.cat([x[0][d: d + n] for x, d, n in zip(want, done, cut)])) < tol
+        done = [d + n for d, n in zip(done, cut)]
+    table, pool = table.cpu(), pool.cpu()
+    for s in range(3):
+        for p in range(total[s]):
+            row = pool[int(table[s, p // page])]
+            k = row[: kv_heads * page * dk].view(kv_heads, page, dk)[:, p % page]
+            v = row[kv_heads * page * dk:].view(kv_heads, page, dv)[:, p % page]
+            assert H.row_error(k, want[s][1][p]) < tol and H.row_error(v, want[s][2][p]) < tol, (s, p)
+        for p in range(max(0, total[s] - (taps - 1)), total[s]):
+            assert torch.equal(ring[ctx.slots[s], p % hist].cpu(), u[s][p, :C].float())
 
 
 @pytest.mark.parametrize("n,experts,top", [(70, 5, 2), (9, 16, 4), (300, 3, 1), (40, 33, 7), (5, 6, 6)])
