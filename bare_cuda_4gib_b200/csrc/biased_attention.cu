@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(512) conv_norm_cache_kernel(const T* __restric
 // registers, PIECES pieces a thread.  With `write_ring` (steps of one token per request only) it also does what
 // conv_ring_write does: the entry it writes is the one the same thread has read as the oldest input.
 template <int TAPS, int PIECES>
-__global__ void __launch_bounds__(PIECES == 1 ? 1024 : 768)
+__global__ void __launch_bounds__(PIECES == 1 ? 768 : 512)
 conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, const float* __restrict__ conv_w,
                            float* __restrict__ ring, const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w,
                            __nv_bfloat16* __restrict__ q_out, PagedCacheKV cache, const int32_t* __restrict__ positions,
@@ -150,62 +150,78 @@ conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
   }
   pdl_wait();
   const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, n_tokens - t0);
+  // where this thread's channels go: 0 q, 1 k, 2 v; its head and the entry in it
+  int kind[PIECES], entry[PIECES], in_head[PIECES], head_of[PIECES];
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    kind[j] = at[j] < qd ? 0 : (at[j] < qd + kd ? 1 : 2);
+    entry[j] = at[j] - (kind[j] == 0 ? 0 : (kind[j] == 1 ? qd : qd + kd));
+    const int dim = kind[j] == 2 ? cache.v_dim : cache.k_dim;
+    head_of[j] = entry[j] / dim;
+    in_head[j] = entry[j] - head_of[j] * dim;
+  }
   int seq = -1;
-  for (int r = 0; r < rows; ++r) {
-    const int t = t0 + r, s = row_seq[t], p = positions[t], parity = r & 1;
-    float* turn = turns + parity * rot_dims;
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)p * inv_freq[i], &turn[half + i], &turn[i]);
-    const bool fresh = s != seq;
-    seq = s;
-    float* ring_slot = ring + (long long)seq_slot[s] * (HIST > 0 ? HIST : 1) * C;
-    float y[PIECES][4];
-    float2 sq = make_float2(0.0f, 0.0f);
+  for (int r0 = 0; r0 < rows; r0 += 4) {      // four rows' inputs are asked for together
+    uint2 in[PIECES][4];
 #pragma unroll
-    for (int j = 0; j < PIECES; ++j) {
-      if (at[j] >= C) continue;
-      if (fresh) conv[j].history(u, u_stride, at[j], t, p, seq_q_start[s], ring_slot, HIST, C);
-      const uint2 now = conv_load4(u + (long long)t * u_stride + at[j]);
-      conv[j].step(now, y[j]);
-      if (HIST > 0 && write_ring) *reinterpret_cast<float4*>(ring_slot + (long long)(p % (HIST > 0 ? HIST : 1)) * C + at[j]) = conv_floats(now);
-      const float e = y[j][0] * y[j][0] + y[j][1] * y[j][1] + y[j][2] * y[j][2] + y[j][3] * y[j][3];
-      if (at[j] < qd) sq.x += e;
-      else if (at[j] < qd + kd) sq.y += e;
-    }
-    sq.x = warp_sum(sq.x);
-    sq.y = warp_sum(sq.y);
-    if (lane == 0) sums[parity][warp] = sq;
-    __syncthreads();      // (two rows' sums and turns in turn: a row's are written again behind the next row's barrier)
-    sq = lane < n_warps ? sums[parity][lane] : make_float2(0.0f, 0.0f);
-    const float rq = 1.0f / sqrtf(warp_sum(sq.x) / (float)qd + eps) * (1.0f + temp_coef * logf((float)((p + 1) / temp_every + 1)));
-    const float rk = 1.0f / sqrtf(warp_sum(sq.y) / (float)kd + eps);
-    const int page = cache_page(cache, s, p), in_page = p % cache.page_tokens;
+    for (int j = 0; j < PIECES; ++j)
+      if (at[j] < C) {
 #pragma unroll
-    for (int j = 0; j < PIECES; ++j) {
-      if (at[j] >= C) continue;
-      __nv_bfloat16* dst;
-      if (at[j] < qd + kd) {
-        const bool is_q = at[j] < qd;
-        const int e = is_q ? at[j] : at[j] - qd, head = e / cache.k_dim, d = e - head * cache.k_dim;
-        const float4 w = *reinterpret_cast<const float4*>((is_q ? q_norm_w : k_norm_w) + e);
-        const float f = is_q ? rq : rk;
-        y[j][0] *= f * w.x; y[j][1] *= f * w.y; y[j][2] *= f * w.z; y[j][3] *= f * w.w;
+        for (int k = 0; k < 4; ++k) in[j][k] = conv_load4(u + (long long)(t0 + min(r0 + k, rows - 1)) * u_stride + at[j]);
+      }
 #pragma unroll
-        for (int x = 0; x < 4; x += 2) {
-          if (d + x < rot_dims) {
-            const float c = turn[(d + x) / 2], sn = turn[half + (d + x) / 2], a = y[j][x], b = y[j][x + 1];
-            y[j][x] = a * c - b * sn;
-            y[j][x + 1] = b * c + a * sn;
+    for (int k = 0; k < 4; ++k) {
+      if (r0 + k >= rows) break;
+      const int t = t0 + r0 + k, s = row_seq[t], p = positions[t], parity = k & 1;
+      float* turn = turns + parity * rot_dims;
+      for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)p * inv_freq[i], &turn[half + i], &turn[i]);
+      const bool fresh = s != seq;
+      seq = s;
+      float* ring_slot = ring + (long long)seq_slot[s] * (HIST > 0 ? HIST : 1) * C;
+      float y[PIECES][4];
+      float2 sq = make_float2(0.0f, 0.0f);
+#pragma unroll
+      for (int j = 0; j < PIECES; ++j) {
+        if (at[j] >= C) continue;
+        if (fresh) conv[j].history(u, u_stride, at[j], t, p, seq_q_start[s], ring_slot, HIST, C);
+        conv[j].step(in[j][k], y[j]);
+        if (HIST > 0 && write_ring) *reinterpret_cast<float4*>(ring_slot + (long long)(p % (HIST > 0 ? HIST : 1)) * C + at[j]) = conv_floats(in[j][k]);
+        const float e = y[j][0] * y[j][0] + y[j][1] * y[j][1] + y[j][2] * y[j][2] + y[j][3] * y[j][3];
+        if (kind[j] == 0) sq.x += e;
+        else if (kind[j] == 1) sq.y += e;
+      }
+      sq.x = warp_sum(sq.x);
+      sq.y = warp_sum(sq.y);
+      if (lane == 0) sums[parity][warp] = sq;
+      __syncthreads();      // (two rows' sums and turns in turn: a row's are written again behind the next row's barrier)
+      sq = lane < n_warps ? sums[parity][lane] : make_float2(0.0f, 0.0f);
+      float rq = 1.0f / sqrtf(warp_sum(sq.x) / (float)qd + eps);
+      const float rk = 1.0f / sqrtf(warp_sum(sq.y) / (float)kd + eps);
+      if (temp_coef != 0.0f) rq *= 1.0f + temp_coef * logf((float)((p + 1) / temp_every + 1));
+      const int page = cache_page(cache, s, p), in_page = p % cache.page_tokens;
+#pragma unroll
+      for (int j = 0; j < PIECES; ++j) {
+        if (at[j] >= C || (kind[j] != 0 && (!write_cache || page < 0))) continue;
+        if (kind[j] != 2) {
+          const float4 w = *reinterpret_cast<const float4*>((kind[j] == 0 ? q_norm_w : k_norm_w) + entry[j]);
+          const float f = kind[j] == 0 ? rq : rk;
+          y[j][0] *= f * w.x; y[j][1] *= f * w.y; y[j][2] *= f * w.z; y[j][3] *= f * w.w;
+#pragma unroll
+          for (int x = 0; x < 4; x += 2) {
+            const int d = in_head[j] + x;
+            if (d < rot_dims) {
+              const float c = turn[d / 2], sn = turn[half + d / 2], e0 = y[j][x], e1 = y[j][x + 1];
+              y[j][x] = e0 * c - e1 * sn;
+              y[j][x + 1] = e1 * c + e0 * sn;
+            }
           }
         }
-        dst = is_q ? q_out + (long long)t * qd + e
-                   : (__nv_bfloat16*)cache.k + (long long)page * cache.page_stride + ((long long)head * cache.page_tokens + in_page) * cache.k_dim + d;
-        if (!is_q && (!write_cache || page < 0)) continue;
-      } else {
-        const int e = at[j] - qd - kd, head = e / cache.v_dim, d = e - head * cache.v_dim;
-        if (!write_cache || page < 0) continue;
-        dst = (__nv_bfloat16*)cache.v + (long long)page * cache.page_stride + ((long long)head * cache.page_tokens + in_page) * cache.v_dim + d;
+        __nv_bfloat16* dst =
+            kind[j] == 0 ? q_out + (long long)t * qd + entry[j]
+                         : (__nv_bfloat16*)(kind[j] == 1 ? cache.k : cache.v) + (long long)page * cache.page_stride +
+                               ((long long)head_of[j] * cache.page_tokens + in_page) * (kind[j] == 1 ? cache.k_dim : cache.v_dim) + in_head[j];
+        *reinterpret_cast<uint2*>(dst) = conv_pack4(y[j]);
       }
-      *reinterpret_cast<uint2*>(dst) = conv_pack4(y[j]);
     }
   }
 }
@@ -230,13 +246,13 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
   const int threads = C >= 2048 ? 512 : (C >= 512 ? 256 : 128);
   PagedCacheKV cache{cache_k, cache_v, block_table, page_stride, table_stride, page_tokens, kv_heads, k_dim, v_dim};
   auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
-  const int pieces = C / 4 <= 1024 ? 1 : 2;
+  const int pieces = C / 4 <= 768 ? 1 : (C / 4 <= 1024 ? 2 : 3);
   const bool vec = dtype == DT_BF16 && taps <= 4 && !(halves && rot_dims) && k_dim % 4 == 0 && v_dim % 4 == 0 &&
-                   C / 4 <= 2 * 768 && u_stride % 4 == 0 && page_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) &&
+                   C / 4 <= 3 * 512 && u_stride % 4 == 0 && page_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) &&
                    aligned(q_norm_w, 16) && aligned(k_norm_w, 16) && aligned(q_out, 8) && aligned(cache_k, 8) && aligned(cache_v, 8);
   if (vec) {
     *ring_written = write_ring;
-    const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 1024 ? 8 : (n_tokens >= 256 ? 2 : 1);
+    const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 512 ? 4 : (n_tokens >= 256 ? 2 : 1);
     const int blocks = (n_tokens + per_block - 1) / per_block;
 #define VEC(TAPS, PIECES)                                                                                              \
   launch_kernel(conv_norm_cache_vec_kernel<TAPS, PIECES>, blocks, wide, (size_t)2 * rot_dims * sizeof(float), stream,  \
@@ -247,7 +263,7 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
   do {                                                                                                                 \
     if (taps == 1) VEC(1, PIECES); else if (taps == 2) VEC(2, PIECES); else if (taps == 3) VEC(3, PIECES); else VEC(4, PIECES); \
   } while (0)
-    if (pieces == 1) TAPS_OF(1); else TAPS_OF(2);
+    if (pieces == 1) TAPS_OF(1); else if (pieces == 2) TAPS_OF(2); else TAPS_OF(3);
 #undef TAPS_OF
 #undef VEC
     return launch_status();

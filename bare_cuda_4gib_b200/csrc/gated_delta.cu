@@ -103,6 +103,8 @@ gated_delta_compact_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
   pdl_wait();
   const int t0 = blockIdx.x * OPER_ROWS, rows = min(OPER_ROWS, n_tokens - t0);
   const int lanes = dk / 4;
+  const bool qk = (blockIdx.y * OPER_THREADS + (threadIdx.x & ~31)) * 4 < 2 * kd;      // the warp has a q or k head
+  const bool first = live && c < 2 * kd && c % dk == 0;
   int seq = -1;
   for (int i0 = 0; i0 < rows; i0 += 4) {      // four rows' inputs are asked for together
     uint2 in[4];
@@ -119,11 +121,14 @@ gated_delta_compact_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
       float y[4];
       conv.step(in[k], y);
 #pragma unroll
-      for (int x = 0; x < 4; ++x) y[x] = __bfloat162float(__float2bfloat16_rn(delta_silu(y[x])));
-      if (live) *reinterpret_cast<uint2*>(compact + (long long)t * C + c) = conv_pack4(y);
-      float sq = y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3];
+      for (int x = 0; x < 4; ++x) y[x] = __fdividef(y[x], 1.0f + __expf(-y[x]));      // silu, to be rounded to bfloat16
+      const uint2 raw = conv_pack4(y);
+      if (live) *reinterpret_cast<uint2*>(compact + (long long)t * C + c) = raw;
+      if (!qk) continue;
+      const float4 r = conv_floats(raw);
+      float sq = r.x * r.x + r.y * r.y + r.z * r.z + r.w * r.w;
       for (int o = lanes >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      if (live && c < 2 * kd && c % dk == 0) lengths[(long long)t * 2 * G + c / dk] = (c < kd ? q_scale : 1.0f) / sqrtf(sq + unit_eps);
+      if (first) lengths[(long long)t * 2 * G + c / dk] = (c < kd ? q_scale : 1.0f) / sqrtf(sq + unit_eps);
     }
   }
 }
@@ -319,7 +324,7 @@ struct DeltaStep {
 };
 
 template <typename T, bool CHANNEL, int CV, int NR>
-__global__ void __launch_bounds__(STEP_THREADS) gated_delta_step_kernel(DeltaStep a, int W) {
+__global__ void __launch_bounds__(STEP_THREADS, NR * CV <= 32 ? 2 : 1) gated_delta_step_kernel(DeltaStep a, int W) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float sm[];
   __shared__ float scratch[32];

@@ -147,10 +147,22 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
     cp_async16(kt + t * LDN + c, src + (in ? G * DK : 0), in);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
-  if (CHANNEL) {
-    for (int e = tid; e < L * DK; e += PREP_THREADS) {
-      const int t = e / DK, i = e % DK;
-      cs[t * LDF + i] = t < count ? delta_log_decay(gates, row0 + t, h * DK + i, neg_a) : 0.0f;
+  if (CHANNEL) {      // a channel per thread, eight tokens' numbers asked for together
+    constexpr int STEP = PREP_THREADS / DK;
+    const int i = tid % DK, first = tid / DK;
+    if (first < STEP) {
+      const float bias = gates.dt_bias[h * DK + i];
+      for (int t0 = first; t0 < L; t0 += 8 * STEP) {
+        float z[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          z[k] = load_any(gates.z, (row0 + min(t0 + k * STEP, count - 1)) * gates.z_stride + h * DK + i, gates.z_dtype);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          const int t = t0 + k * STEP;
+          if (t < L) cs[t * LDF + i] = t < count ? neg_a * delta_softplus(z[k] + bias) : 0.0f;
+        }
+      }
     }
   } else if (tid < L) {
     cs[tid] = tid < count ? delta_log_decay(gates, row0 + tid, h, neg_a) : 0.0f;
@@ -505,13 +517,14 @@ struct WalkShared {
   static constexpr size_t BYTES = 2 * (size_t)(6 * L * LDN + 2 * L * LDP + 2 * DK * LDC + 2 * L * LDC) + 4 * DK;
 };
 
-// A block's warps: WARPS of them per group of 16 value columns.
+// A block's warps, WARPS of them per group of 16 value columns in each of two roles: the first half makes U and carries
+// the state, the second half makes the outputs.
 template <int PC>
-__global__ void __launch_bounds__(WARPS * 2 * PC)
+__global__ void __launch_bounds__(WARPS * 4 * PC)
 gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__ out, const int32_t* __restrict__ seq_slot,
                         const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_q_len, int H, int dv) {
   pdl_launch_dependents();
-  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 2 * PC;
+  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 4 * PC;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* Ws = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2][L][LDN]: rounded, rest (and so on below)
   __nv_bfloat16* Qs = Ws + 2 * L * LDN;
@@ -526,7 +539,8 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
   if (q_len <= 0) return;
   const int q_start = seq_q_start[seq];
   const int warp = (threadIdx.x >> 5) % WARPS, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3, mid = lane >> 3;
-  const int own = (threadIdx.x >> 5) / WARPS * 16, col0 = blockIdx.x * PC + own;      // this warp's 16 columns
+  const bool carries = threadIdx.x < THREADS / 2;
+  const int own = (threadIdx.x >> 5) / WARPS % (PC / 16) * 16, col0 = blockIdx.x * PC + own;      // this warp's 16 columns
   Ss += own;
   Us += own;
   float* S_g = state + (((long long)seq_slot[seq] * H + h) * DK) * dv + col0;
@@ -588,7 +602,7 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
   };
   load_wq(0);
   load_pk(0);
-  load_u(0);
+  if (carries) load_u(0);
 
   float sreg[MTW][NT][4];      // the state's tiles this warp owns, float32, for the whole walk
   auto keep_state = [&]() {    // ... and as the products' operand in shared memory
@@ -608,119 +622,104 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
         }
     }
   };
+  if (carries) {
 #pragma unroll
-  for (int i = 0; i < MTW; ++i) {
-    const int mt = warp + i * WARPS;
+    for (int i = 0; i < MTW; ++i) {
+      const int mt = warp + i * WARPS;
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
+      for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const float2 v = mt < MT_N ? *reinterpret_cast<const float2*>(S_g + (long long)(mt * 16 + gq + r * 8) * dv + nt * 8 + tq * 2)
-                                   : make_float2(0.0f, 0.0f);
-        sreg[i][nt][r * 2] = v.x;
-        sreg[i][nt][r * 2 + 1] = v.y;
-      }
+        for (int r = 0; r < 2; ++r) {
+          const float2 v = mt < MT_N ? *reinterpret_cast<const float2*>(S_g + (long long)(mt * 16 + gq + r * 8) * dv + nt * 8 + tq * 2)
+                                     : make_float2(0.0f, 0.0f);
+          sreg[i][nt][r * 2] = v.x;
+          sreg[i][nt][r * 2 + 1] = v.y;
+        }
+    }
+    keep_state();
   }
-  keep_state();
   asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
 
   for (int ch = 0; ch < n_chunks; ++ch) {
     const int count = min(L, q_len - ch * L);
     const long long row0 = q_start + (long long)ch * L;
-    // ---- U = T V - W S and O = Q' S, this warp's 16 tokens
-    float ws[NT][4] = {}, acc[NT][4] = {};
+    // ---- W S (for U = T V - W S) or Q' S (the outputs' first part), this warp's 16 tokens and 16 columns
+    float acc[NT][4] = {};
+    const __nv_bfloat16* As = carries ? Ws : Qs;
 #pragma unroll
     for (int s = 0; s < DK / 16; ++s) {
-      uint32_t wh[4], wl[4], qh[4], ql[4];
+      uint32_t ah[4], al[4], sh[4], sl[4];
       const int at = (warp * 16 + (lane & 15)) * LDN + s * 16 + (lane >> 4) * 8;
-      ldmatrix_x4(wh, Ws + at);
-      ldmatrix_x4(wl, Ws + L * LDN + at);
-      ldmatrix_x4(qh, Qs + at);
-      ldmatrix_x4(ql, Qs + L * LDN + at);
+      ldmatrix_x4(ah, As + at);
+      ldmatrix_x4(al, As + L * LDN + at);
+      const int sat = (s * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (mid >> 1) * 8;
+      ldmatrix_x4_trans(sh, Ss + sat);
+      ldmatrix_x4_trans(sl, Ss + DK * LDC + sat);
 #pragma unroll
-      for (int nt = 0; nt < NT; nt += 2) {
-        uint32_t sh[4], sl[4];
-        const int sat = (s * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (nt + (mid >> 1)) * 8;
-        ldmatrix_x4_trans(sh, Ss + sat);
-        ldmatrix_x4_trans(sl, Ss + DK * LDC + sat);
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          mma_bf16(ws[nt + x], wh, sh[x * 2], sh[x * 2 + 1]);
-          mma_bf16(acc[nt + x], qh, sh[x * 2], sh[x * 2 + 1]);
-          mma_bf16(ws[nt + x], wl, sh[x * 2], sh[x * 2 + 1]);
-          mma_bf16(acc[nt + x], ql, sh[x * 2], sh[x * 2 + 1]);
-          mma_bf16(ws[nt + x], wh, sl[x * 2], sl[x * 2 + 1]);
-          mma_bf16(acc[nt + x], qh, sl[x * 2], sl[x * 2 + 1]);
-        }
-      }
+      for (int x = 0; x < 2; ++x) mma_split(acc[x], ah, al, sh[x * 2], sh[x * 2 + 1], sl[x * 2], sl[x * 2 + 1]);
     }
+    if (carries) {
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
+      for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        uint32_t hi, lo;
-        split2(u0[nt][r * 2] - ws[nt][r * 2], u0[nt][r * 2 + 1] - ws[nt][r * 2 + 1], hi, lo);
-        const int at = (warp * 16 + gq + r * 8) * LDC + nt * 8 + tq * 2;
-        *reinterpret_cast<uint32_t*>(Us + at) = hi;
-        *reinterpret_cast<uint32_t*>(Us + L * LDC + at) = lo;
-      }
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          split2(u0[nt][r * 2] - acc[nt][r * 2], u0[nt][r * 2 + 1] - acc[nt][r * 2 + 1], hi, lo);
+          const int at = (warp * 16 + gq + r * 8) * LDC + nt * 8 + tq * 2;
+          *reinterpret_cast<uint32_t*>(Us + at) = hi;
+          *reinterpret_cast<uint32_t*>(Us + L * LDC + at) = lo;
+        }
+    }
     asm volatile("cp.async.wait_group 0;" ::: "memory");      // this chunk's P and K''
     __syncthreads();      // U is whole; every warp has read the old state, W and Q'
     load_wq(ch + 1);
-    load_u(ch + 1);
+    if (carries) {
+      load_u(ch + 1);
 #pragma unroll
-    for (int i = 0; i < MTW; ++i) {
-      const int mt = warp + i * WARPS;
-      if (mt >= MT_N) break;
-      const float e0 = ends[mt * 16 + gq], e1 = ends[mt * 16 + gq + 8];
+      for (int i = 0; i < MTW; ++i) {
+        const int mt = warp + i * WARPS;
+        if (mt >= MT_N) break;
+        const float e0 = ends[mt * 16 + gq], e1 = ends[mt * 16 + gq + 8];
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        sreg[i][nt][0] *= e0; sreg[i][nt][1] *= e0;
-        sreg[i][nt][2] *= e1; sreg[i][nt][3] *= e1;
+        for (int nt = 0; nt < NT; ++nt) {
+          sreg[i][nt][0] *= e0; sreg[i][nt][1] *= e0;
+          sreg[i][nt][2] *= e1; sreg[i][nt][3] *= e1;
+        }
       }
     }
-    // ---- O += P U and S <- diag(exp(c_last)) S + K''^T U
+    // ---- S <- diag(exp(c_last)) S + K''^T U, or the outputs' second part, P U
 #pragma unroll
     for (int kk = 0; kk < L / 16; ++kk) {
-      uint32_t uh[NT / 2][4], ul[NT / 2][4];
+      if (!carries && kk > warp) break;
+      uint32_t uh[4], ul[4];
+      const int uat = (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (mid >> 1) * 8;
+      ldmatrix_x4_trans(uh, Us + uat);
+      ldmatrix_x4_trans(ul, Us + L * LDC + uat);
+      if (carries) {
 #pragma unroll
-      for (int nt = 0; nt < NT; nt += 2) {
-        const int at = (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (nt + (mid >> 1)) * 8;
-        ldmatrix_x4_trans(uh[nt / 2], Us + at);
-        ldmatrix_x4_trans(ul[nt / 2], Us + L * LDC + at);
-      }
-      if (kk <= warp) {
+        for (int i = 0; i < MTW; ++i) {
+          const int mt = warp + i * WARPS;
+          if (mt >= MT_N) break;
+          uint32_t kh[4], kl[4];      // K''^T as the row operand: the stored [token][channel] tile, transposed on the way in
+          const int at = (kk * 16 + (mid >> 1) * 8 + (lane & 7)) * LDN + mt * 16 + (mid & 1) * 8;
+          ldmatrix_x4_trans(kh, Ks + at);
+          ldmatrix_x4_trans(kl, Ks + L * LDN + at);
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) mma_split(sreg[i][nt], kh, kl, uh[nt * 2], uh[nt * 2 + 1], ul[nt * 2], ul[nt * 2 + 1]);
+        }
+      } else {
         uint32_t ph[4], pl[4];
         const int at = (warp * 16 + (lane & 15)) * LDP + kk * 16 + (lane >> 4) * 8;
         ldmatrix_x4(ph, Ps + at);
         ldmatrix_x4(pl, Ps + L * LDP + at);
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt) {
-          const int f = nt / 2, x = (nt & 1) * 2;
-          mma_bf16(acc[nt], ph, uh[f][x], uh[f][x + 1]);
-          mma_bf16(acc[nt], pl, uh[f][x], uh[f][x + 1]);
-          mma_bf16(acc[nt], ph, ul[f][x], ul[f][x + 1]);
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < MTW; ++i) {
-        const int mt = warp + i * WARPS;
-        if (mt >= MT_N) break;
-        uint32_t kh[4], kl[4];      // K''^T as the row operand: the stored [token][channel] tile, transposed on the way in
-        const int at = (kk * 16 + (mid >> 1) * 8 + (lane & 7)) * LDN + mt * 16 + (mid & 1) * 8;
-        ldmatrix_x4_trans(kh, Ks + at);
-        ldmatrix_x4_trans(kl, Ks + L * LDN + at);
-#pragma unroll
-        for (int nt = 0; nt < NT; ++nt) {
-          const int f = nt / 2, x = (nt & 1) * 2;
-          mma_bf16(sreg[i][nt], kh, uh[f][x], uh[f][x + 1]);
-          mma_bf16(sreg[i][nt], kl, uh[f][x], uh[f][x + 1]);
-          mma_bf16(sreg[i][nt], kh, ul[f][x], ul[f][x + 1]);
-        }
+        for (int nt = 0; nt < NT; ++nt) mma_split(acc[nt], ph, pl, uh[nt * 2], uh[nt * 2 + 1], ul[nt * 2], ul[nt * 2 + 1]);
       }
     }
-    {
+    if (carries) {
+      keep_state();
+    } else {
       const int t = warp * 16 + gq;
       float* dst = out + (row0 + t) * ((long long)H * dv) + (long long)h * dv + col0 + tq * 2;
 #pragma unroll
@@ -730,11 +729,11 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
           if (t + r * 8 < count)
             *reinterpret_cast<float2*>(dst + (long long)r * 8 * H * dv + nt * 8) = make_float2(acc[nt][r * 2], acc[nt][r * 2 + 1]);
     }
-    keep_state();
     asm volatile("cp.async.wait_group 0;" ::: "memory");      // the next chunk's W and Q'
     __syncthreads();      // the new state is whole; every warp has read P, K'' and U
     load_pk(ch + 1);
   }
+  if (!carries) return;
 #pragma unroll
   for (int i = 0; i < MTW; ++i) {
     const int mt = warp + i * WARPS;
@@ -804,7 +803,7 @@ extern "C" int llm_gated_delta_walk(const void* w, const void* q, const void* k,
         return launch_status();                                                                                         \
       configured = true;                                                                                                \
     }                                                                                                                   \
-    launch_kernel(gated_delta_walk_kernel<PC>, grid, WARPS * 2 * PC, smem, stream, in, state, out, seq_slot, seq_q_start,      \
+    launch_kernel(gated_delta_walk_kernel<PC>, grid, WARPS * 4 * PC, smem, stream, in, state, out, seq_slot, seq_q_start,      \
                   seq_q_len, heads, dv);                                                                                \
   } while (0)
   if (columns == 16) GO(16); else GO(32);

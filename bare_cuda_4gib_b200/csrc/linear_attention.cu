@@ -601,15 +601,15 @@ template <typename TG, int PIECES>
 __global__ void __launch_bounds__(256)
 gated_group_norm_vec_kernel(const float* __restrict__ x, const TG* __restrict__ gate, long long gate_stride,
                             const float* __restrict__ weight, int weight_len, __nv_bfloat16* __restrict__ out,
-                            long long out_stride, int rows, int channels, int group, int lanes, int gate_kind, float eps,
+                            long long out_stride, int channels, int group, int lane_bits, int gate_kind, float eps,
                             float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
-  const int groups = channels / group, lane = threadIdx.x % lanes;
-  const bool live = item < (long long)rows * groups;
-  const long long r = live ? item / groups : 0;
-  const int g = live ? (int)(item - r * groups) : 0;
+  const int lanes = 1 << lane_bits, groups = channels / group, lane = threadIdx.x & (lanes - 1);
+  const int item = (blockIdx.x * blockDim.x + threadIdx.x) >> lane_bits;      // group of the row; grid (groups, rows)
+  const bool live = item < groups;
+  const long long r = blockIdx.y;
+  const int g = live ? item : 0;
   float4 v[PIECES], z[PIECES];
   float sq = 0.0f;
 #pragma unroll
@@ -622,11 +622,11 @@ gated_group_norm_vec_kernel(const float* __restrict__ x, const TG* __restrict__ 
   for (int o = lanes >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
   const float scale = out_scale / sqrtf(sq / (float)group + eps);
   if (!live) return;
-  auto act = [&](float a) { return gate_kind == GATE_SILU ? a / (1.0f + expf(-a)) : 1.0f / (1.0f + expf(-a)); };
+  auto act = [&](float a) { return (gate_kind == GATE_SILU ? a : 1.0f) * (1.0f / (1.0f + __expf(-a))); };
 #pragma unroll
   for (int j = 0; j < PIECES; ++j) {
     const int c = g * group + (lane + j * lanes) * 4;
-    const float4 w = *reinterpret_cast<const float4*>(weight + c % weight_len);
+    const float4 w = *reinterpret_cast<const float4*>(weight + (weight_len == group ? c - g * group : c % weight_len));
     const __nv_bfloat162 lo = __floats2bfloat162_rn(v[j].x * scale * w.x * act(z[j].x), v[j].y * scale * w.y * act(z[j].y));
     const __nv_bfloat162 hi = __floats2bfloat162_rn(v[j].z * scale * w.z * act(z[j].z), v[j].w * scale * w.w * act(z[j].w));
     uint2 raw;
@@ -647,15 +647,17 @@ extern "C" int llm_gated_group_norm(const float* x, const void* gate, int gate_d
   const bool wide = group >= 512;
   auto at = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
   const int gbytes = gate_dtype == DT_BF16 ? 8 : 16;
-  if (out_dtype == DT_BF16 && group >= 8 && group <= 1024 && (group & (group - 1)) == 0 && weight_len % 4 == 0 &&
+  if (out_dtype == DT_BF16 && rows <= 65535 && group >= 8 && group <= 1024 && (group & (group - 1)) == 0 && weight_len % 4 == 0 &&
       gate_stride % 4 == 0 && out_stride % 4 == 0 && at(x, 16) && at(gate, gbytes) && at(weight, 16) && at(out, 8) &&
       (gate_dtype == DT_F32 || gate_dtype == DT_BF16)) {
     const int lanes = group / 4 < 32 ? group / 4 : 32, pieces = group / 4 / lanes;
-    const long long threads = items * lanes;
-    const unsigned grid = (unsigned)((threads + 255) / 256);
+    int lane_bits = 0;
+    while ((1 << lane_bits) < lanes) ++lane_bits;
+    const int threads = (channels / group) * lanes, block = threads >= 256 ? 256 : (threads + 31) / 32 * 32;
+    const dim3 grid((threads + block - 1) / block, rows);
 #define VEC(TG, PIECES)                                                                                               \
-  launch_kernel(gated_group_norm_vec_kernel<TG, PIECES>, grid, 256, 0, stream, x, (const TG*)gate, gate_stride, weight, \
-                weight_len, (__nv_bfloat16*)out, out_stride, rows, channels, group, lanes, gate_kind, eps, out_scale)
+  launch_kernel(gated_group_norm_vec_kernel<TG, PIECES>, grid, block, 0, stream, x, (const TG*)gate, gate_stride, weight, \
+                weight_len, (__nv_bfloat16*)out, out_stride, channels, group, lane_bits, gate_kind, eps, out_scale)
 #define PIECES_OF(TG)                                                                                                 \
   do {                                                                                                                \
     if (pieces == 1) VEC(TG, 1); else if (pieces == 2) VEC(TG, 2); else if (pieces == 4) VEC(TG, 4); else VEC(TG, 8);   \

@@ -5,6 +5,8 @@
 
 #include "common.cuh"
 
+#include <string.h>
+
 // four bfloat16 numbers as they lie in memory, and as floats
 __device__ __forceinline__ uint2 conv_load4(const __nv_bfloat16* p) { return *reinterpret_cast<const uint2*>(p); }
 __device__ __forceinline__ float4 conv_floats(uint2 raw) {
@@ -12,7 +14,10 @@ __device__ __forceinline__ float4 conv_floats(uint2 raw) {
                      __uint_as_float(raw.y & 0xffff0000u));
 }
 __device__ __forceinline__ uint32_t conv_pack2(float lo, float hi) {
-  return (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(lo)) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(hi)) << 16);
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  uint32_t raw;
+  memcpy(&raw, &v, 4);
+  return raw;
 }
 __device__ __forceinline__ uint2 conv_pack4(const float (&y)[4]) { return make_uint2(conv_pack2(y[0], y[1]), conv_pack2(y[2], y[3])); }
 
