@@ -136,9 +136,9 @@ conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
                            float eps, float temp_coef, int temp_every, int write_cache, int write_ring,
                            const float* __restrict__ inv_freq, int rot_dims) {
   pdl_launch_dependents();
-  extern __shared__ float turns[];             // [2][rot_dims] cosines, then sines, of two rows in turn
-  __shared__ float2 sums[2][32];
-  constexpr int HIST = TAPS - 1;
+  constexpr int HIST = TAPS - 1, BATCH = PIECES == 1 ? 4 : 2;
+  extern __shared__ float turns[];             // [BATCH][rot_dims] cosines, then sines, of a batch of rows
+  __shared__ float2 sums[BATCH][32];
   const int C = qd + kd + vd, half = rot_dims / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n_warps = blockDim.x >> 5;
   ConvColumns<TAPS> conv[PIECES];
@@ -161,40 +161,51 @@ conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
     in_head[j] = entry[j] - head_of[j] * dim;
   }
   int seq = -1;
-  for (int r0 = 0; r0 < rows; r0 += 4) {      // four rows' inputs are asked for together
-    uint2 in[PIECES][4];
+  for (int r0 = 0; r0 < rows; r0 += BATCH) {      // some rows' inputs are asked for together
+    uint2 in[PIECES][BATCH];
 #pragma unroll
     for (int j = 0; j < PIECES; ++j)
       if (at[j] < C) {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) in[j][k] = conv_load4(u + (long long)(t0 + min(r0 + k, rows - 1)) * u_stride + at[j]);
+        for (int k = 0; k < BATCH; ++k) in[j][k] = conv_load4(u + (long long)(t0 + min(r0 + k, rows - 1)) * u_stride + at[j]);
       }
+    const int batch = min(BATCH, rows - r0);
+    for (int i = threadIdx.x; i < batch * half; i += blockDim.x) {
+      const int k = i / half, x = i - k * half;
+      sincosf((float)positions[t0 + r0 + k] * inv_freq[x], &turns[k * rot_dims + half + x], &turns[k * rot_dims + x]);
+    }
+    float y[BATCH][PIECES][4];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      if (r0 + k >= rows) break;
-      const int t = t0 + r0 + k, s = row_seq[t], p = positions[t], parity = k & 1;
-      float* turn = turns + parity * rot_dims;
-      for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)p * inv_freq[i], &turn[half + i], &turn[i]);
-      const bool fresh = s != seq;
-      seq = s;
-      float* ring_slot = ring + (long long)seq_slot[s] * (HIST > 0 ? HIST : 1) * C;
-      float y[PIECES][4];
+    for (int k = 0; k < BATCH; ++k) {
       float2 sq = make_float2(0.0f, 0.0f);
+      if (k < batch) {
+        const int t = t0 + r0 + k, s = row_seq[t], p = positions[t];
+        const bool fresh = s != seq;
+        seq = s;
+        float* ring_slot = ring + (long long)seq_slot[s] * (HIST > 0 ? HIST : 1) * C;
 #pragma unroll
-      for (int j = 0; j < PIECES; ++j) {
-        if (at[j] >= C) continue;
-        if (fresh) conv[j].history(u, u_stride, at[j], t, p, seq_q_start[s], ring_slot, HIST, C);
-        conv[j].step(in[j][k], y[j]);
-        if (HIST > 0 && write_ring) *reinterpret_cast<float4*>(ring_slot + (long long)(p % (HIST > 0 ? HIST : 1)) * C + at[j]) = conv_floats(in[j][k]);
-        const float e = y[j][0] * y[j][0] + y[j][1] * y[j][1] + y[j][2] * y[j][2] + y[j][3] * y[j][3];
-        if (kind[j] == 0) sq.x += e;
-        else if (kind[j] == 1) sq.y += e;
+        for (int j = 0; j < PIECES; ++j) {
+          if (at[j] >= C) continue;
+          if (fresh) conv[j].history(u, u_stride, at[j], t, p, seq_q_start[s], ring_slot, HIST, C);
+          conv[j].step(in[j][k], y[k][j]);
+          if (HIST > 0 && write_ring)
+            *reinterpret_cast<float4*>(ring_slot + (long long)(p % (HIST > 0 ? HIST : 1)) * C + at[j]) = conv_floats(in[j][k]);
+          const float e = y[k][j][0] * y[k][j][0] + y[k][j][1] * y[k][j][1] + y[k][j][2] * y[k][j][2] + y[k][j][3] * y[k][j][3];
+          if (kind[j] == 0) sq.x += e;
+          else if (kind[j] == 1) sq.y += e;
+        }
+        sq.x = warp_sum(sq.x);
+        sq.y = warp_sum(sq.y);
       }
-      sq.x = warp_sum(sq.x);
-      sq.y = warp_sum(sq.y);
-      if (lane == 0) sums[parity][warp] = sq;
-      __syncthreads();      // (two rows' sums and turns in turn: a row's are written again behind the next row's barrier)
-      sq = lane < n_warps ? sums[parity][lane] : make_float2(0.0f, 0.0f);
+      if (lane == 0) sums[k][warp] = sq;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < BATCH; ++k) {
+      if (k >= batch) break;
+      const int t = t0 + r0 + k, s = row_seq[t], p = positions[t];
+      const float* turn = turns + k * rot_dims;
+      const float2 sq = lane < n_warps ? sums[k][lane] : make_float2(0.0f, 0.0f);
       float rq = 1.0f / sqrtf(warp_sum(sq.x) / (float)qd + eps);
       const float rk = 1.0f / sqrtf(warp_sum(sq.y) / (float)kd + eps);
       if (temp_coef != 0.0f) rq *= 1.0f + temp_coef * logf((float)((p + 1) / temp_every + 1));
@@ -202,17 +213,18 @@ conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
 #pragma unroll
       for (int j = 0; j < PIECES; ++j) {
         if (at[j] >= C || (kind[j] != 0 && (!write_cache || page < 0))) continue;
+        float v[4] = {y[k][j][0], y[k][j][1], y[k][j][2], y[k][j][3]};
         if (kind[j] != 2) {
           const float4 w = *reinterpret_cast<const float4*>((kind[j] == 0 ? q_norm_w : k_norm_w) + entry[j]);
           const float f = kind[j] == 0 ? rq : rk;
-          y[j][0] *= f * w.x; y[j][1] *= f * w.y; y[j][2] *= f * w.z; y[j][3] *= f * w.w;
+          v[0] *= f * w.x; v[1] *= f * w.y; v[2] *= f * w.z; v[3] *= f * w.w;
 #pragma unroll
           for (int x = 0; x < 4; x += 2) {
             const int d = in_head[j] + x;
             if (d < rot_dims) {
-              const float c = turn[d / 2], sn = turn[half + d / 2], e0 = y[j][x], e1 = y[j][x + 1];
-              y[j][x] = e0 * c - e1 * sn;
-              y[j][x + 1] = e1 * c + e0 * sn;
+              const float c = turn[d / 2], sn = turn[half + d / 2], e0 = v[x], e1 = v[x + 1];
+              v[x] = e0 * c - e1 * sn;
+              v[x + 1] = e1 * c + e0 * sn;
             }
           }
         }
@@ -220,9 +232,10 @@ conv_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ u, long long u_stri
             kind[j] == 0 ? q_out + (long long)t * qd + entry[j]
                          : (__nv_bfloat16*)(kind[j] == 1 ? cache.k : cache.v) + (long long)page * cache.page_stride +
                                ((long long)head_of[j] * cache.page_tokens + in_page) * (kind[j] == 1 ? cache.k_dim : cache.v_dim) + in_head[j];
-        *reinterpret_cast<uint2*>(dst) = conv_pack4(y[j]);
+        *reinterpret_cast<uint2*>(dst) = conv_pack4(v);
       }
     }
+    __syncthreads();      // sums and turns have been read
   }
 }
 
@@ -248,14 +261,14 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
   auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
   const int pieces = C / 4 <= 768 ? 1 : (C / 4 <= 1024 ? 2 : 3);
   const bool vec = dtype == DT_BF16 && taps <= 4 && !(halves && rot_dims) && k_dim % 4 == 0 && v_dim % 4 == 0 &&
-                   C / 4 <= 3 * 512 && u_stride % 4 == 0 && page_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) &&
+                   C / 4 <= 3 * 512 && u_stride % 4 == 0 && page_stride % 4 == 0 && aligned(u, 8) && aligned(conv_w, 16) && aligned(ring, 16) &&
                    aligned(q_norm_w, 16) && aligned(k_norm_w, 16) && aligned(q_out, 8) && aligned(cache_k, 8) && aligned(cache_v, 8);
   if (vec) {
     *ring_written = write_ring;
     const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 512 ? 4 : (n_tokens >= 256 ? 2 : 1);
     const int blocks = (n_tokens + per_block - 1) / per_block;
 #define VEC(TAPS, PIECES)                                                                                              \
-  launch_kernel(conv_norm_cache_vec_kernel<TAPS, PIECES>, blocks, wide, (size_t)2 * rot_dims * sizeof(float), stream,  \
+  launch_kernel(conv_norm_cache_vec_kernel<TAPS, PIECES>, blocks, wide, (size_t)4 * rot_dims * sizeof(float), stream,  \
                 (const __nv_bfloat16*)u, u_stride, conv_w, ring, q_norm_w, k_norm_w, (__nv_bfloat16*)q_out, cache,      \
                 positions, row_seq, seq_slot, seq_q_start, n_tokens, per_block, qd, kd, vd, eps, temp_coef, temp_every, \
                 write_cache, write_ring, inv_freq, rot_dims)

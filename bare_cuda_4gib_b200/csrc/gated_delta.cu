@@ -145,7 +145,7 @@ extern "C" int llm_gated_delta_operands(const void* u, int dtype, long long u_st
   LLM_HOST_CHECK(smem <= 200 * 1024, ERR_BAD_SIZE);
   auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
   if (compact && dtype == DT_BF16 && taps <= 4 && dk >= 16 && dk <= 128 && (dk & (dk - 1)) == 0 && dv % 4 == 0 &&
-      u_stride % 4 == 0 && aligned(u, 8) && aligned(ring, 16) && aligned(compact, 8)) {
+      u_stride % 4 == 0 && aligned(u, 8) && aligned(conv_w, 16) && aligned(ring, 16) && aligned(compact, 8)) {
     const int C = 2 * kv_heads * dk + heads * dv;
     const dim3 grid((n_tokens + OPER_ROWS - 1) / OPER_ROWS, (C / 4 + OPER_THREADS - 1) / OPER_THREADS);
 #define COMPACT(TAPS)                                                                                                 \

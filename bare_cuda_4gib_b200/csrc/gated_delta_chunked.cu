@@ -250,7 +250,7 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
           const int t = t0 + (f & 1) * 8, c = s * 16 + tq * 2 + (f >> 1) * 8;
           const float2 k2 = pair_of(kt + t * LDN + c), q2 = pair_of(qt + t * LDN + c);
           const float2 ct = *reinterpret_cast<const float2*>(cs + t * LDF + c);
-          const float e0 = exp2f(ct.x - r[f >> 1].x), e1 = exp2f(ct.y - r[f >> 1].y);
+          const float e0 = exp2_ftz(ct.x - r[f >> 1].x), e1 = exp2_ftz(ct.y - r[f >> 1].y);
           split2(k2.x * e0, k2.y * e1, kh[f], kl[f]);
           split2(q2.x * e0, q2.y * e1, qh[f], ql[f]);
         }
@@ -261,7 +261,7 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
           for (int f = 0; f < 2; ++f) {
             const int j = 16 * b + nt * 8 + gq, c = s * 16 + tq * 2 + f * 8;
             const float2 k2 = pair_of(kt + j * LDN + c), cj = *reinterpret_cast<const float2*>(cs + j * LDF + c);
-            split2(k2.x * exp2f(r[f].x - cj.x), k2.y * exp2f(r[f].y - cj.y), bh[f], bl[f]);
+            split2(k2.x * exp2_ftz(r[f].x - cj.x), k2.y * exp2_ftz(r[f].y - cj.y), bh[f], bl[f]);
           }
           mma_split(kk[nt], kh, kl, bh[0], bh[1], bl[0], bl[1]);
           mma_split(qk[nt], qh, ql, bh[0], bh[1], bl[0], bl[1]);
@@ -276,7 +276,7 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
           if (j > t) continue;
           float x = 0.0f, y = 0.0f;
           for (int i = 0; i < DK; ++i) {
-            const float f = __bfloat162float(kt[j * LDN + i]) * exp2f(cs[t * LDF + i] - cs[j * LDF + i]);
+            const float f = __bfloat162float(kt[j * LDN + i]) * exp2_ftz(cs[t * LDF + i] - cs[j * LDF + i]);
             x = fmaf(__bfloat162float(kt[t * LDN + i]), f, x);
             y = fmaf(__bfloat162float(qt[t * LDN + i]), f, y);
           }
@@ -292,7 +292,7 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
         float pv[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float f = j + e <= t ? (CHANNEL ? 1.0f : exp2f(cs[t] - cs[j + e])) * k_len[j + e] : 0.0f;
+          const float f = j + e <= t ? (CHANNEL ? 1.0f : exp2_ftz(cs[t] - cs[j + e])) * k_len[j + e] : 0.0f;
           pv[e] = j + e <= t ? qk[nt][r * 2 + e] * q_len_[t] * f : 0.0f;
           Lm[t * LDL + j + e] = j + e < t ? betas[t] * k_len[t] * kk[nt][r * 2 + e] * f : 0.0f;
         }
@@ -321,8 +321,8 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
 #pragma unroll
       for (int y = 0; y < 2; ++y) {
         const float ct = CHANNEL ? cs[t * LDF + c + 2 * x + y] : cs[t];
-        f[y] = exp2f(ct);
-        last[y] = exp2f((CHANNEL ? cs[(L - 1) * LDF + c + 2 * x + y] : cs[L - 1]) - ct);
+        f[y] = exp2_ftz(ct);
+        last[y] = exp2_ftz((CHANNEL ? cs[(L - 1) * LDF + c + 2 * x + y] : cs[L - 1]) - ct);
       }
       split2(k2.x * kn * f[0], k2.y * kn * f[1], hd[x], ld[x]);
       split2(q2.x * qn * f[0], q2.y * qn * f[1], hq[x], lq[x]);
@@ -339,7 +339,7 @@ gated_delta_prepare_kernel(const __nv_bfloat16* __restrict__ qkv, const float* _
     }
   }
   if (tid < DK)
-    o.end[chunk_id(q_start, seq, chunk) * ((long long)H * DK) + h * DK + tid] = exp2f(CHANNEL ? cs[(L - 1) * LDF + tid] : cs[L - 1]);
+    o.end[chunk_id(q_start, seq, chunk) * ((long long)H * DK) + h * DK + tid] = exp2_ftz(CHANNEL ? cs[(L - 1) * LDF + tid] : cs[L - 1]);
   // ---- (1 + L)^-1, the blocks on the diagonal by substitution, a lane per column ...
   if (warp >= PREP_THREADS / 32 - 4 && lane < 16) {
     const int a = warp - (PREP_THREADS / 32 - 4);
@@ -512,27 +512,29 @@ constexpr int MT_N = DK / 16;                     // row tiles of the state
 constexpr int MTW = (MT_N + WARPS - 1) / WARPS;   // of which a warp owns at most this many
 
 template <int PC>
-struct WalkShared {
+struct WalkShared {      // two chunks' W, K'' and decays; one's Q' and P; the state and U as operands
   static constexpr int LDC = PC + 8;
-  static constexpr size_t BYTES = 2 * (size_t)(6 * L * LDN + 2 * L * LDP + 2 * DK * LDC + 2 * L * LDC) + 4 * DK;
+  static constexpr size_t BYTES = 2 * (size_t)(10 * L * LDN + 2 * L * LDP + 2 * DK * LDC + 2 * L * LDC) + 2 * 4 * DK;
 };
 
 // A block's warps, WARPS of them per group of 16 value columns in each of two roles: the first half makes U and carries
-// the state, the second half makes the outputs.
+// the state, the second half makes the outputs.  A chunk's W and K'' arrive by cp.async while the chunk before it is
+// worked on, Q' and P (which the state does not wait for) as soon as their one place is free; T V is read straight into
+// the registers that need it, one chunk ahead.
 template <int PC>
 __global__ void __launch_bounds__(WARPS * 4 * PC)
 gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__ out, const int32_t* __restrict__ seq_slot,
                         const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_q_len, int H, int dv) {
   pdl_launch_dependents();
-  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 4 * PC;
+  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 4 * PC, KS = DK / 16;
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  __nv_bfloat16* Ws = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2][L][LDN]: rounded, rest (and so on below)
-  __nv_bfloat16* Qs = Ws + 2 * L * LDN;
-  __nv_bfloat16* Ks = Qs + 2 * L * LDN;
-  __nv_bfloat16* Ps = Ks + 2 * L * LDN;                                // [2][L][LDP]
+  __nv_bfloat16* W0 = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2 chunks][2][L][LDN]: rounded, rest (and so on below)
+  __nv_bfloat16* K0 = W0 + 4 * L * LDN;                                // [2 chunks][2][L][LDN]
+  __nv_bfloat16* Qs = K0 + 4 * L * LDN;                                // [2][L][LDN]
+  __nv_bfloat16* Ps = Qs + 2 * L * LDN;                                // [2][L][LDP]
   __nv_bfloat16* Ss = Ps + 2 * L * LDP;                                // [2][DK][LDC]
   __nv_bfloat16* Us = Ss + 2 * DK * LDC;                               // [2][L][LDC]
-  float* ends = reinterpret_cast<float*>(Us + 2 * L * LDC);            // [DK]
+  float* ends0 = reinterpret_cast<float*>(Us + 2 * L * LDC);           // [2 chunks][DK]
   pdl_wait();
   const int h = blockIdx.y, seq = blockIdx.z;
   const int q_len = seq_q_len[seq];
@@ -546,47 +548,46 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
   float* S_g = state + (((long long)seq_slot[seq] * H + h) * DK) * dv + col0;
   const int n_chunks = (q_len + L - 1) / L;
 
-  constexpr int CN = DK / 8;
-  auto load_wq = [&](int ch) {
-    if (ch < n_chunks) {
-      const int count = min(L, q_len - ch * L);
-      const long long row0 = q_start + (long long)ch * L;
-      for (int i = threadIdx.x; i < L * CN; i += THREADS) {
-        const int r = i / CN, c = (i % CN) * 8;
-        const bool valid = r < count;
-        const long long src = valid ? (row0 + r) * ((long long)H * DK) + h * DK + c : 0;
-        cp_async16(Ws + r * LDN + c, in.w + src, valid);
-        cp_async16(Ws + (L + r) * LDN + c, in.w + in.hl + src, valid);
-        cp_async16(Qs + r * LDN + c, in.q + src, valid);
-        cp_async16(Qs + (L + r) * LDN + c, in.q + in.hl + src, valid);
-      }
+  // rows of one chunk's tile of `in` (both parts), zero behind the request's last token
+  auto load_tile = [&](__nv_bfloat16* dst, const __nv_bfloat16* from, int ch) {
+    constexpr int CN = DK / 8;
+    const int count = min(L, q_len - ch * L);
+    const long long row0 = q_start + (long long)ch * L;
+    for (int i = threadIdx.x; i < L * CN; i += THREADS) {
+      const int r = i / CN, c = (i % CN) * 8;
+      const bool valid = r < count;
+      const long long src = valid ? (row0 + r) * ((long long)H * DK) + h * DK + c : 0;
+      cp_async16(dst + r * LDN + c, from + src, valid);
+      cp_async16(dst + (L + r) * LDN + c, from + in.hl + src, valid);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  auto load_pk = [&](int ch) {
+  auto load_wk = [&](int ch) {
     if (ch < n_chunks) {
-      const int count = min(L, q_len - ch * L);
-      const long long row0 = q_start + (long long)ch * L;
-      for (int i = threadIdx.x; i < L * CN; i += THREADS) {
-        const int r = i / CN, c = (i % CN) * 8;
-        const bool valid = r < count;
-        const long long src = valid ? (row0 + r) * ((long long)H * DK) + h * DK + c : 0;
-        cp_async16(Ks + r * LDN + c, in.k + src, valid);
-        cp_async16(Ks + (L + r) * LDN + c, in.k + in.hl + src, valid);
-      }
-      for (int i = threadIdx.x; i < L * (L / 8); i += THREADS) {
-        const int r = i / (L / 8), c = (i % (L / 8)) * 8;
-        const bool valid = r < count;
-        const long long src = valid ? (row0 + r) * ((long long)H * L) + h * L + c : 0;
-        cp_async16(Ps + r * LDP + c, in.p + src, valid);
-        cp_async16(Ps + (L + r) * LDP + c, in.p + in.p_hl + src, valid);
-      }
+      const int st = ch & 1;
+      load_tile(W0 + st * 2 * L * LDN, in.w, ch);
+      load_tile(K0 + st * 2 * L * LDN, in.k, ch);
       const float* end = in.end + chunk_id(q_start, seq, ch) * ((long long)H * DK) + h * DK;
-      for (int i = threadIdx.x; i < DK / 4; i += THREADS) cp_async16(ends + i * 4, end + i * 4, true);
+      for (int i = threadIdx.x; i < DK / 4; i += THREADS) cp_async16(ends0 + st * DK + i * 4, end + i * 4, true);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float u0[NT][4];      // T V of this warp's rows, asked for one chunk ahead
+  auto load_q = [&](int ch) {
+    if (ch < n_chunks) load_tile(Qs, in.q, ch);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  auto load_p = [&](int ch) {
+    const int count = min(L, q_len - ch * L);
+    const long long row0 = q_start + (long long)ch * L;
+    for (int i = threadIdx.x; i < L * (L / 8); i += THREADS) {
+      const int r = i / (L / 8), c = (i % (L / 8)) * 8;
+      const bool valid = r < count;
+      const long long src = valid ? (row0 + r) * ((long long)H * L) + h * L + c : 0;
+      cp_async16(Ps + r * LDP + c, in.p + src, valid);
+      cp_async16(Ps + (L + r) * LDP + c, in.p + in.p_hl + src, valid);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float u0[NT][4];      // (carries) T V of this warp's rows
   auto load_u = [&](int ch) {
     const int count = ch < n_chunks ? min(L, q_len - ch * L) : 0;
     const int t = warp * 16 + gq;
@@ -600,11 +601,10 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
         u0[nt][r * 2 + 1] = v.y;
       }
   };
-  load_wq(0);
-  load_pk(0);
-  if (carries) load_u(0);
+  load_wk(0);
+  load_q(0);
 
-  float sreg[MTW][NT][4];      // the state's tiles this warp owns, float32, for the whole walk
+  float sreg[MTW][NT][4];      // (carries) the state's tiles this warp owns, float32, for the whole walk
   auto keep_state = [&]() {    // ... and as the products' operand in shared memory
 #pragma unroll
     for (int i = 0; i < MTW; ++i) {
@@ -623,6 +623,7 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
     }
   };
   if (carries) {
+    load_u(0);
 #pragma unroll
     for (int i = 0; i < MTW; ++i) {
       const int mt = warp + i * WARPS;
@@ -638,17 +639,21 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
     }
     keep_state();
   }
-  asm volatile("cp.async.wait_group 1;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
 
   for (int ch = 0; ch < n_chunks; ++ch) {
-    const int count = min(L, q_len - ch * L);
+    const int count = min(L, q_len - ch * L), st = ch & 1;
     const long long row0 = q_start + (long long)ch * L;
+    const __nv_bfloat16 *Ws = W0 + st * 2 * L * LDN, *Ks = K0 + st * 2 * L * LDN;
+    const float* ends = ends0 + st * DK;
+    load_p(ch);
+    load_wk(ch + 1);      // into the other set, which every warp left at the last chunk's end
     // ---- W S (for U = T V - W S) or Q' S (the outputs' first part), this warp's 16 tokens and 16 columns
     float acc[NT][4] = {};
     const __nv_bfloat16* As = carries ? Ws : Qs;
 #pragma unroll
-    for (int s = 0; s < DK / 16; ++s) {
+    for (int s = 0; s < KS; ++s) {
       uint32_t ah[4], al[4], sh[4], sl[4];
       const int at = (warp * 16 + (lane & 15)) * LDN + s * 16 + (lane >> 4) * 8;
       ldmatrix_x4(ah, As + at);
@@ -670,12 +675,13 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
           *reinterpret_cast<uint32_t*>(Us + at) = hi;
           *reinterpret_cast<uint32_t*>(Us + L * LDC + at) = lo;
         }
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");      // this chunk's P and K''
-    __syncthreads();      // U is whole; every warp has read the old state, W and Q'
-    load_wq(ch + 1);
-    if (carries) {
       load_u(ch + 1);
+    }
+    asm volatile("cp.async.wait_group 1;" ::: "memory");      // this chunk's P
+    __syncthreads();      // U is whole; every warp has read the old state and Q'
+    load_q(ch + 1);
+    // ---- S <- diag(exp(c_last)) S + K''^T U, or the outputs' second part, P U
+    if (carries) {
 #pragma unroll
       for (int i = 0; i < MTW; ++i) {
         const int mt = warp + i * WARPS;
@@ -688,7 +694,6 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
         }
       }
     }
-    // ---- S <- diag(exp(c_last)) S + K''^T U, or the outputs' second part, P U
 #pragma unroll
     for (int kk = 0; kk < L / 16; ++kk) {
       if (!carries && kk > warp) break;
@@ -729,9 +734,8 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
           if (t + r * 8 < count)
             *reinterpret_cast<float2*>(dst + (long long)r * 8 * H * dv + nt * 8) = make_float2(acc[nt][r * 2], acc[nt][r * 2 + 1]);
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");      // the next chunk's W and Q'
-    __syncthreads();      // the new state is whole; every warp has read P, K'' and U
-    load_pk(ch + 1);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");      // the next chunk's W, K'' and Q'
+    __syncthreads();      // the new state is whole; every warp has read this chunk's tiles and U
   }
   if (!carries) return;
 #pragma unroll

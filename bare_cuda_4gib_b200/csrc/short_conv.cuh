@@ -26,12 +26,17 @@ struct ConvColumns {
   float w[4][TAPS];
   uint2 v[TAPS > 1 ? TAPS - 1 : 1];      // inputs of positions p - TAPS + 1 .. p - 1
 
-  // conv_w [channels][TAPS] float32, c the first of the four channels
+  // conv_w [channels][TAPS] float32, 16-byte aligned; c the first of the four channels
   __device__ __forceinline__ void load_weights(const float* conv_w, int c) {
+    const float4* src = reinterpret_cast<const float4*>(conv_w + (long long)c * TAPS);      // 4 TAPS numbers, 16-byte aligned
 #pragma unroll
-    for (int x = 0; x < 4; ++x)
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) w[x][j] = conv_w[(long long)(c + x) * TAPS + j];
+    for (int i = 0; i < TAPS; ++i) {
+      const float4 f = src[i];
+      w[(4 * i) / TAPS][(4 * i) % TAPS] = f.x;
+      w[(4 * i + 1) / TAPS][(4 * i + 1) % TAPS] = f.y;
+      w[(4 * i + 2) / TAPS][(4 * i + 2) % TAPS] = f.z;
+      w[(4 * i + 3) / TAPS][(4 * i + 3) % TAPS] = f.w;
+    }
   }
 
   // The inputs ahead of row t, at position p of a request whose rows start at `q_start`: the step's own rows, the
