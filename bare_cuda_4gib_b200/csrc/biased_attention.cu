@@ -265,7 +265,7 @@ extern "C" int llm_conv_norm_cache(const void* u, int dtype, long long u_stride,
                    aligned(q_norm_w, 16) && aligned(k_norm_w, 16) && aligned(q_out, 8) && aligned(cache_k, 8) && aligned(cache_v, 8);
   if (vec) {
     *ring_written = write_ring;
-    const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 512 ? 4 : (n_tokens >= 256 ? 2 : 1);
+    const int wide = ((C / 4 + pieces - 1) / pieces + 31) / 32 * 32, per_block = n_tokens >= 512 ? ((n_tokens + 147) / 148 + 3) / 4 * 4 : (n_tokens >= 256 ? 2 : 1);
     const int blocks = (n_tokens + per_block - 1) / per_block;
 #define VEC(TAPS, PIECES)                                                                                              \
   launch_kernel(conv_norm_cache_vec_kernel<TAPS, PIECES>, blocks, wide, (size_t)4 * rot_dims * sizeof(float), stream,  \

@@ -517,16 +517,16 @@ struct WalkShared {      // two chunks' W, K'' and decays; one's Q' and P; the s
   static constexpr size_t BYTES = 2 * (size_t)(10 * L * LDN + 2 * L * LDP + 2 * DK * LDC + 2 * L * LDC) + 2 * 4 * DK;
 };
 
-// A block's warps, WARPS of them per group of 16 value columns in each of two roles: the first half makes U and carries
+// A block's warps, WARPS of them in each of two roles and every one with all PC columns: the first half makes U and carries
 // the state, the second half makes the outputs.  A chunk's W and K'' arrive by cp.async while the chunk before it is
 // worked on, Q' and P (which the state does not wait for) as soon as their one place is free; T V is read straight into
 // the registers that need it, one chunk ahead.
 template <int PC>
-__global__ void __launch_bounds__(WARPS * 4 * PC)
+__global__ void __launch_bounds__(WARPS * 64)
 gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__ out, const int32_t* __restrict__ seq_slot,
                         const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_q_len, int H, int dv) {
   pdl_launch_dependents();
-  constexpr int LDC = WalkShared<PC>::LDC, NT = 2, THREADS = WARPS * 4 * PC, KS = DK / 16;
+  constexpr int LDC = WalkShared<PC>::LDC, NT = PC / 8, THREADS = WARPS * 64, KS = DK / 16;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* W0 = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2 chunks][2][L][LDN]: rounded, rest (and so on below)
   __nv_bfloat16* K0 = W0 + 4 * L * LDN;                                // [2 chunks][2][L][LDN]
@@ -542,9 +542,7 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
   const int q_start = seq_q_start[seq];
   const int warp = (threadIdx.x >> 5) % WARPS, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3, mid = lane >> 3;
   const bool carries = threadIdx.x < THREADS / 2;
-  const int own = (threadIdx.x >> 5) / WARPS % (PC / 16) * 16, col0 = blockIdx.x * PC + own;      // this warp's 16 columns
-  Ss += own;
-  Us += own;
+  const int col0 = blockIdx.x * PC;
   float* S_g = state + (((long long)seq_slot[seq] * H + h) * DK) * dv + col0;
   const int n_chunks = (q_len + L - 1) / L;
 
@@ -649,20 +647,24 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
     const float* ends = ends0 + st * DK;
     load_p(ch);
     load_wk(ch + 1);      // into the other set, which every warp left at the last chunk's end
-    // ---- W S (for U = T V - W S) or Q' S (the outputs' first part), this warp's 16 tokens and 16 columns
+    // ---- W S (for U = T V - W S) or Q' S (the outputs' first part), this warp's 16 tokens
     float acc[NT][4] = {};
     const __nv_bfloat16* As = carries ? Ws : Qs;
 #pragma unroll
     for (int s = 0; s < KS; ++s) {
-      uint32_t ah[4], al[4], sh[4], sl[4];
+      uint32_t ah[4], al[4];
       const int at = (warp * 16 + (lane & 15)) * LDN + s * 16 + (lane >> 4) * 8;
       ldmatrix_x4(ah, As + at);
       ldmatrix_x4(al, As + L * LDN + at);
-      const int sat = (s * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (mid >> 1) * 8;
-      ldmatrix_x4_trans(sh, Ss + sat);
-      ldmatrix_x4_trans(sl, Ss + DK * LDC + sat);
 #pragma unroll
-      for (int x = 0; x < 2; ++x) mma_split(acc[x], ah, al, sh[x * 2], sh[x * 2 + 1], sl[x * 2], sl[x * 2 + 1]);
+      for (int nt = 0; nt < NT; nt += 2) {
+        uint32_t sh[4], sl[4];
+        const int sat = (s * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (nt + (mid >> 1)) * 8;
+        ldmatrix_x4_trans(sh, Ss + sat);
+        ldmatrix_x4_trans(sl, Ss + DK * LDC + sat);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) mma_split(acc[nt + x], ah, al, sh[x * 2], sh[x * 2 + 1], sl[x * 2], sl[x * 2 + 1]);
+      }
     }
     if (carries) {
 #pragma unroll
@@ -697,10 +699,13 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
 #pragma unroll
     for (int kk = 0; kk < L / 16; ++kk) {
       if (!carries && kk > warp) break;
-      uint32_t uh[4], ul[4];
-      const int uat = (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (mid >> 1) * 8;
-      ldmatrix_x4_trans(uh, Us + uat);
-      ldmatrix_x4_trans(ul, Us + L * LDC + uat);
+      uint32_t uh[NT / 2][4], ul[NT / 2][4];
+#pragma unroll
+      for (int nt = 0; nt < NT; nt += 2) {
+        const int uat = (kk * 16 + (mid & 1) * 8 + (lane & 7)) * LDC + (nt + (mid >> 1)) * 8;
+        ldmatrix_x4_trans(uh[nt / 2], Us + uat);
+        ldmatrix_x4_trans(ul[nt / 2], Us + L * LDC + uat);
+      }
       if (carries) {
 #pragma unroll
         for (int i = 0; i < MTW; ++i) {
@@ -711,7 +716,10 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
           ldmatrix_x4_trans(kh, Ks + at);
           ldmatrix_x4_trans(kl, Ks + L * LDN + at);
 #pragma unroll
-          for (int nt = 0; nt < NT; ++nt) mma_split(sreg[i][nt], kh, kl, uh[nt * 2], uh[nt * 2 + 1], ul[nt * 2], ul[nt * 2 + 1]);
+          for (int nt = 0; nt < NT; ++nt) {
+            const uint32_t *h2 = uh[nt / 2] + (nt & 1) * 2, *l2 = ul[nt / 2] + (nt & 1) * 2;
+            mma_split(sreg[i][nt], kh, kl, h2[0], h2[1], l2[0], l2[1]);
+          }
         }
       } else {
         uint32_t ph[4], pl[4];
@@ -719,7 +727,10 @@ gated_delta_walk_kernel(Tiles in, float* __restrict__ state, float* __restrict__
         ldmatrix_x4(ph, Ps + at);
         ldmatrix_x4(pl, Ps + L * LDP + at);
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt) mma_split(acc[nt], ph, pl, uh[nt * 2], uh[nt * 2 + 1], ul[nt * 2], ul[nt * 2 + 1]);
+        for (int nt = 0; nt < NT; ++nt) {
+          const uint32_t *h2 = uh[nt / 2] + (nt & 1) * 2, *l2 = ul[nt / 2] + (nt & 1) * 2;
+          mma_split(acc[nt], ph, pl, h2[0], h2[1], l2[0], l2[1]);
+        }
       }
     }
     if (carries) {
@@ -807,7 +818,7 @@ extern "C" int llm_gated_delta_walk(const void* w, const void* q, const void* k,
         return launch_status();                                                                                         \
       configured = true;                                                                                                \
     }                                                                                                                   \
-    launch_kernel(gated_delta_walk_kernel<PC>, grid, WARPS * 4 * PC, smem, stream, in, state, out, seq_slot, seq_q_start,      \
+    launch_kernel(gated_delta_walk_kernel<PC>, grid, WARPS * 64, smem, stream, in, state, out, seq_slot, seq_q_start,      \
                   seq_q_len, heads, dv);                                                                                \
   } while (0)
   if (columns == 16) GO(16); else GO(32);
