@@ -47,13 +47,13 @@ __device__ __forceinline__ float lane_dot(const T* __restrict__ x, const TW* __r
   return dot;
 }
 
-template <typename T, typename TW>
+// CHOSEN: weights from the softmax over the chosen experts' logits
+template <typename T, typename TW, bool CHOSEN>
 __global__ void __launch_bounds__(MOE_ROUTE_WARPS * 32)
 moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restrict__ w_router,
                  const TW* __restrict__ w_shared_gate, int hidden, int experts, int top, float router_scale,
                  int32_t* __restrict__ ids, float* __restrict__ weights, float* __restrict__ shared_gate, int n_tokens,
-                 const float* __restrict__ correction, int groups, int keep, const float* __restrict__ bias,
-                 int chosen_softmax) {
+                 const float* __restrict__ correction, int groups, int keep, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   // a block per token: its warps share the experts' dot products (and the shared gate's, counted as one
@@ -75,7 +75,7 @@ moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restri
   __syncthreads();
   if (warp != 0) return;
   float sum = 1.0f;
-  if (!chosen_softmax) {      // otherwise the score stays the logit, and the weights are made after the choice
+  if (!CHOSEN) {      // otherwise the score stays the logit, and the weights are made after the choice
     float mx = -INFINITY;
     for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, s[e]);
     mx = warp_max(mx);
@@ -140,11 +140,11 @@ moe_route_kernel(const T* __restrict__ h, long long h_stride, const TW* __restri
       ids[(long long)t * top + k] = at;
       weights[(long long)t * top + k] = s[at] * router_scale;
       choice[at] = -INFINITY;
-      group_best[k] = s[at];      // (the groups' values are no longer needed: the chosen ones' scores in order)
+      if (CHOSEN) group_best[k] = s[at];      // (the groups' values are no longer needed: the chosen ones' scores in order)
     }
     __syncwarp();
   }
-  if (chosen_softmax) {
+  if (CHOSEN) {
     float mx = -INFINITY;
     for (int k = lane; k < top; k += 32) mx = fmaxf(mx, group_best[k]);
     mx = warp_max(mx);
@@ -164,15 +164,17 @@ extern "C" int llm_moe_route(const void* h, int dtype, long long h_stride, const
   LLM_HOST_CHECK(groups <= 1 || (experts % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (experts / groups)),
                  ERR_BAD_SIZE);
   const int blocks = n_tokens;
-#define ROUTE(T, TW)                                                                                                 \
-  launch_kernel(moe_route_kernel<T, TW>, blocks, MOE_ROUTE_WARPS * 32, 0, stream, (const T*)h, h_stride,              \
+#define ROUTE(T, TW) (chosen_softmax ? ROUTE_AS(T, TW, true) : ROUTE_AS(T, TW, false))
+#define ROUTE_AS(T, TW, CHOSEN)                                                                                      \
+  launch_kernel(moe_route_kernel<T, TW, CHOSEN>, blocks, MOE_ROUTE_WARPS * 32, 0, stream, (const T*)h, h_stride,              \
                 (const TW*)w_router, (const TW*)w_shared_gate, hidden, experts, top, router_scale, ids, weights,        \
-                shared_gate, n_tokens, correction, groups, keep, bias, chosen_softmax)
+                shared_gate, n_tokens, correction, groups, keep, bias)
   if (dtype == DT_F32 && w_dtype == DT_F32) ROUTE(float, float);
   else if (dtype == DT_BF16 && w_dtype == DT_BF16) ROUTE(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == DT_BF16 && w_dtype == DT_F32) ROUTE(__nv_bfloat16, float);
   else return ERR_BAD_DTYPE;
 #undef ROUTE
+#undef ROUTE_AS
   return launch_status();
 }
 
